@@ -24,12 +24,13 @@ def register_cache_kind(kind: str, first_needed: Callable[["CacheNeed", int], in
 class CacheNeed:
     """Keys and values per position: `kind` says which positions must be kept ("full": all;
     "window": the last `window`; "chunk": the chunk of `window` positions the next query lies in; or a registered kind
-    of the mixer's own)."""
+    of the mixer's own). `keep`: a sequence's first positions that are kept whatever the kind gives back."""
     kind: str
     kv_heads: int
     head_dim: int
     window: int | None = None
     v_dim: int | None = None      # width of a value head where it differs from the keys' (None: head_dim)
+    keep: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -40,9 +41,17 @@ class CacheNeed:
             raise ValueError(f"cache kind {self.kind!r}; known: {', '.join(sorted(CACHE_KINDS))}")
         if (self.kind in ("window", "chunk")) != (self.window is not None) and self.kind in ("full", "window", "chunk"):
             raise ValueError("a window or chunk cache needs its size, a full cache has none")
+        if self.keep < 0:
+            raise ValueError(f"a cache that keeps the first {self.keep} positions")
 
     def first_needed(self, length: int) -> int:
         return CACHE_KINDS[self.kind](self, length)
+
+    def pages_seen(self) -> int | None:
+        """The most pages one query can see (None: no bound but its sequence)."""
+        if self.window is None or self.kind not in ("window", "chunk"):
+            return None
+        return (self.window + 2 * PAGE - 2) // PAGE + (self.keep + PAGE - 1) // PAGE
 
 
 register_cache_kind("full", lambda need, length: 0)

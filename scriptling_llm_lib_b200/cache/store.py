@@ -52,13 +52,14 @@ class KVGroup:
             lst.append(self.pool.alloc())
 
     def release_unseen(self, slot: int, length: int) -> None:
-        """Give back the pages no query at a position >= length can see (the need's kind says which)."""
+        """Give back the pages no query at a position >= length can see (the need's kind says which; pages that hold one of
+        the kept first positions stay)."""
         first_seen = self.need.first_needed(length)
         if first_seen <= 0:
             return
         lst = self.pages[slot]
         for i, pg in enumerate(lst):
-            if pg >= 0 and (i + 1) * PAGE - 1 < first_seen:
+            if pg >= 0 and (i + 1) * PAGE - 1 < first_seen and i * PAGE >= self.need.keep:
                 self.pool.free(pg)
                 lst[i] = -1
 

@@ -1,5 +1,6 @@
 // Causal attention of a prompt step over the paged cache for key and value widths the tcgen05 kernels do not take
-// (keys KD wide, values VD wide, each a multiple of 16 out of a short list; storage rows may be wider). bfloat16 operands on
+// (keys KD wide, values VD wide, each a multiple of 16 out of a short list; heads narrower than that, in multiples of 8, are
+// filled up with zeros on the chip, and storage rows may be wider). bfloat16 operands on
 // mma.sync.m16n8k16 with float accumulation, scores, cap, softmax statistics and sink in float; the weights enter the
 // product with the values rounded to bfloat16, as in the library's other tensor-core attention kernels.
 //
@@ -18,7 +19,7 @@
 struct PmArgs {
   const bf16* q;        // [T, q_ld]; head h at columns h * q_hw, its first KD columns used
   int q_ld, q_hw;
-  bf16* out;            // [T, out_ld]; head h at columns h * o_hw: VD columns written, the rest of the head's o_hw set to 0
+  bf16* out;            // [T, out_ld]; head h at columns h * o_hw: vd columns written, the rest of the head's o_hw set to 0
   int out_ld, o_hw;
   const int* seq_start; // [B + 1]
   const int* seq_pos0;  // [B]
@@ -27,9 +28,12 @@ struct PmArgs {
   const bf16* kpages;   // [pages][G][64][k_w]
   const bf16* vpages;   // [pages][G][64][v_w]
   int k_w, v_w;
-  int H, G, window;
+  int kd, vd;           // the widths used: at most KD and VD, multiples of 8
+  int H, G, window, keep;
   float scale, softcap;
   const float* sink;    // [H] or null
+  const bf16* gate;     // null, or [T, gate_ld]: the output's elements are multiplied by the sigmoid of its columns h * vd + d
+  int gate_ld;
 };
 
 __device__ __forceinline__ void pm_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -70,14 +74,15 @@ __global__ void __launch_bounds__(128) attn_prefill_mma_kernel(PmArgs p) {
 #pragma unroll
     for (int kk = 0; kk < KD / 16; kk++) {
       const int c = kk * 16 + 2 * t;
-      qa[kk][0] = ra < S ? *(const uint32_t*)(qa_row + c) : 0u;
-      qa[kk][1] = rb < S ? *(const uint32_t*)(qb_row + c) : 0u;
-      qa[kk][2] = ra < S ? *(const uint32_t*)(qa_row + c + 8) : 0u;
-      qa[kk][3] = rb < S ? *(const uint32_t*)(qb_row + c + 8) : 0u;
+      const bool lo = c < p.kd, hi = c + 8 < p.kd;
+      qa[kk][0] = ra < S && lo ? *(const uint32_t*)(qa_row + c) : 0u;
+      qa[kk][1] = rb < S && lo ? *(const uint32_t*)(qb_row + c) : 0u;
+      qa[kk][2] = ra < S && hi ? *(const uint32_t*)(qa_row + c + 8) : 0u;
+      qa[kk][3] = rb < S && hi ? *(const uint32_t*)(qb_row + c + 8) : 0u;
     }
   }
   const int k_hi = pos0 + r0 + nq;                                   // one past the last key any query of the block sees
-  const int t_lo = first_seen(pos0 + r0, p.window) / PM_BK, t_hi = (k_hi - 1) / PM_BK;
+  const SeenKeys seen_keys(pos0 + r0, k_hi - 1, p.window, p.keep);   // a tile is a page
 
   auto load_tile = [&](int stage, int tile) {
     bf16* ks = pm_sm + (size_t)stage * (KT + VT);
@@ -88,13 +93,13 @@ __global__ void __launch_bounds__(128) attn_prefill_mma_kernel(PmArgs p) {
     const bf16* vp = p.vpages + base * p.v_w;
     for (int e = tid; e < PM_BK * (KD / 8); e += 128) {
       const int kk = e / (KD / 8), c = (e % (KD / 8)) * 8;
-      if (page >= 0 && tile * PM_BK + kk < k_hi) pm_cp16(ks + kk * KS + c, kp + (size_t)kk * p.k_w + c);
+      if (page >= 0 && tile * PM_BK + kk < k_hi && c < p.kd) pm_cp16(ks + kk * KS + c, kp + (size_t)kk * p.k_w + c);
       else *(uint4*)(ks + kk * KS + c) = make_uint4(0, 0, 0, 0);
     }
     for (int e = tid; e < PM_BK * (VD / 8); e += 128) {
       const int kk = e / (VD / 8), c = (e % (VD / 8)) * 8;
       // rows past the last key hold whatever the page held before: their weights are 0, but 0 * NaN is NaN
-      if (page >= 0 && tile * PM_BK + kk < k_hi) pm_cp16(vs + kk * VS + c, vp + (size_t)kk * p.v_w + c);
+      if (page >= 0 && tile * PM_BK + kk < k_hi && c < p.vd) pm_cp16(vs + kk * VS + c, vp + (size_t)kk * p.v_w + c);
       else *(uint4*)(vs + kk * VS + c) = make_uint4(0, 0, 0, 0);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -109,11 +114,11 @@ __global__ void __launch_bounds__(128) attn_prefill_mma_kernel(PmArgs p) {
   const float sc = p.softcap > 0.f ? p.scale / p.softcap : p.scale * PM_LOG2E;
   const float cap_l2 = p.softcap * PM_LOG2E;
 
-  load_tile(0, t_lo);
-  for (int tile = t_lo; tile <= t_hi; tile++) {
-    const int stage = (tile - t_lo) & 1;
-    if (tile < t_hi) {
-      load_tile(stage ^ 1, tile + 1);
+  load_tile(0, seen_keys.page(0));
+  for (int v = 0; v < seen_keys.pages; v++) {
+    const int tile = seen_keys.page(v), stage = v & 1;
+    if (v + 1 < seen_keys.pages) {
+      load_tile(stage ^ 1, seen_keys.page(v + 1));
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -145,7 +150,7 @@ __global__ void __launch_bounds__(128) attn_prefill_mma_kernel(PmArgs p) {
           const int qpos = c < 2 ? qpos0 : qpos1, first = c < 2 ? first0 : first1;
           float v = s[nb][c] * sc;
           if (p.softcap > 0.f) v = cap_l2 * tanhf(v);
-          v = (key <= qpos && key >= first) ? v : -INFINITY;
+          v = key_seen(key, qpos, first, p.keep) ? v : -INFINITY;
           s[nb][c] = v;
           if (c < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
         }
@@ -200,12 +205,23 @@ __global__ void __launch_bounds__(128) attn_prefill_mma_kernel(PmArgs p) {
   const int ra = r0 + warp * 16 + g, rb = ra + 8;
   bf16* oa = p.out + (size_t)(row0 + ra) * p.out_ld + (size_t)h * p.o_hw;
   bf16* ob = p.out + (size_t)(row0 + rb) * p.out_ld + (size_t)h * p.o_hw;
+  if (p.gate != nullptr) {
+    const bf16* ga = p.gate + (size_t)(row0 + ra) * p.gate_ld + (size_t)h * p.vd;
+    const bf16* gb = ga + (size_t)8 * p.gate_ld;
+#pragma unroll
+    for (int i = 0; i < VD / 8; i++) {
+      const int c = i * 8 + 2 * t;
+      if (c < p.vd && ra < S) { o[i][0] *= sigmoid_of(to_f32(ga[c])); o[i][1] *= sigmoid_of(to_f32(ga[c + 1])); }
+      if (c < p.vd && rb < S) { o[i][2] *= sigmoid_of(to_f32(gb[c])); o[i][3] *= sigmoid_of(to_f32(gb[c + 1])); }
+    }
+  }
 #pragma unroll
   for (int i = 0; i < VD / 8; i++) {
-    if (ra < S) *(uint32_t*)(oa + i * 8 + 2 * t) = pm_pack(o[i][0] * i0, o[i][1] * i0);
-    if (rb < S) *(uint32_t*)(ob + i * 8 + 2 * t) = pm_pack(o[i][2] * i1, o[i][3] * i1);
+    const int c = i * 8 + 2 * t;
+    if (c < p.vd && ra < S) *(uint32_t*)(oa + c) = pm_pack(o[i][0] * i0, o[i][1] * i0);
+    if (c < p.vd && rb < S) *(uint32_t*)(ob + c) = pm_pack(o[i][2] * i1, o[i][3] * i1);
   }
-  for (int c = VD + 2 * t; c < p.o_hw; c += 8) {       // the head's columns past the values (a padded layout): zeros
+  for (int c = p.vd + 2 * t; c < p.o_hw; c += 8) {       // the head's columns past the values (a padded layout): zeros
     if (ra < S) *(uint32_t*)(oa + c) = 0u;
     if (rb < S) *(uint32_t*)(ob + c) = 0u;
   }
@@ -225,9 +241,13 @@ static int pm_launch(const PmArgs& a, int B, int max_new, cudaStream_t stream) {
   SLLM_RETURN_LAST();
 }
 
-// The key widths and value widths the kernel is built for; a caller pads its rows with zeros up to the next one.
+// The widths the kernel takes: what a head lacks to the next key and value width it is built for is zeros on the chip.
 SLLM_EXPORT int sllm_attn_prefill_mma_takes(int kd, int vd) {
-  return (kd == 64 || kd == 96 || kd == 128 || kd == 192 || kd == 256) && (vd == 64 || vd == 128);
+  return kd >= 8 && kd <= 256 && kd % 8 == 0 && vd >= 8 && vd <= 128 && vd % 8 == 0;
+}
+static int pm_built_for(int w, bool keys) {
+  if (keys) return w <= 64 ? 64 : w <= 96 ? 96 : w <= 128 ? 128 : w <= 192 ? 192 : 256;
+  return w <= 32 ? 32 : w <= 64 ? 64 : 128;
 }
 
 // q [T, q_ld] with head h at columns h * q_hw; out [T, out_ld] with head h at columns h * o_hw; kpages [pages][G][64][k_w],
@@ -236,16 +256,20 @@ SLLM_EXPORT int sllm_attn_prefill_mma_takes(int kd, int vd) {
 SLLM_EXPORT int sllm_attn_prefill_mma_bf16(const void* q, int q_ld, int q_hw, void* out, int out_ld, int o_hw, const int* seq_start,
                                            const int* seq_pos0, const int* block_table, int max_pages, const void* kpages, int k_w,
                                            const void* vpages, int v_w, int B, int max_new, int H, int G, int kd, int vd, int window,
-                                           float scale, float softcap, const float* sink, cudaStream_t stream) {
+                                           int keep, float scale, float softcap, const float* sink, const void* gate, int gate_ld,
+                                           cudaStream_t stream) {
   if (B <= 0 || max_new <= 0) return 0;
-  if (!sllm_attn_prefill_mma_takes(kd, vd) || G < 1 || H % G != 0 || kd > q_hw || kd > k_w || vd > v_w || vd > o_hw ||
+  if (!sllm_attn_prefill_mma_takes(kd, vd) || keep < 0 || G < 1 || H % G != 0 || kd > q_hw || kd > k_w || vd > v_w || vd > o_hw ||
+      (gate && gate_ld < H * vd) ||
       ((q_ld | q_hw | out_ld | o_hw | k_w | v_w) & 7) || (((uintptr_t)q | (uintptr_t)out | (uintptr_t)kpages | (uintptr_t)vpages) & 15))
     return SLLM_ERR_ARG;
   PmArgs a{(const bf16*)q, q_ld, q_hw, (bf16*)out, out_ld, o_hw, seq_start, seq_pos0, block_table, max_pages, (const bf16*)kpages,
-           (const bf16*)vpages, k_w, v_w, H, G, window, scale, softcap, sink};
-#define PM_CASE(K, V) if (kd == K && vd == V) return pm_launch<K, V>(a, B, max_new, stream)
-  PM_CASE(64, 64); PM_CASE(64, 128); PM_CASE(96, 64); PM_CASE(96, 128); PM_CASE(128, 64); PM_CASE(128, 128);
-  PM_CASE(192, 64); PM_CASE(192, 128); PM_CASE(256, 64); PM_CASE(256, 128);
+           (const bf16*)vpages, k_w, v_w, kd, vd, H, G, window, keep, scale, softcap, sink, (const bf16*)gate, gate_ld};
+  const int K0 = pm_built_for(kd, true), V0 = pm_built_for(vd, false);
+#define PM_CASE(K, V) if (K0 == K && V0 == V) return pm_launch<K, V>(a, B, max_new, stream)
+  PM_CASE(64, 32); PM_CASE(64, 64); PM_CASE(64, 128); PM_CASE(96, 32); PM_CASE(96, 64); PM_CASE(96, 128);
+  PM_CASE(128, 32); PM_CASE(128, 64); PM_CASE(128, 128); PM_CASE(192, 32); PM_CASE(192, 64); PM_CASE(192, 128);
+  PM_CASE(256, 32); PM_CASE(256, 64); PM_CASE(256, 128);
 #undef PM_CASE
   return SLLM_ERR_ARG;
 }

@@ -48,18 +48,20 @@ struct FtArgs {
   const int* seq_pos0;  // [B]
   const int* block_table;
   int max_pages;
-  int H, G, window;
+  int H, G, window, keep;
   float scale;
   int* err;
   int n_qt, n_seqs, n_items;   // query tiles per sequence (of the longest), sequences, work items
   int pair_heads;              // pair kernel: 1: an item is heads 2i, 2i+1 on one query tile; 0: query tiles 2i, 2i+1 of one head
   float softcap;               // > 0: a score s (scaled) becomes softcap * tanh(s / softcap) before the softmax
   const float* sink;           // [H] or null: exp(sink[h]) joins head h's denominator, with no key and no value
+  const bf16* gate;            // null, or [T, gate_ld]: output element (h, d) is multiplied by the sigmoid of column h * hd + d
+  int gate_ld;
 };
 
 // What a block works on in its r-th round.
 struct FtItem {
-  int b, h, g, row0, r0, nq, pos0, t_lo, t_hi, n_tiles, q_hi;
+  int b, h, g, row0, r0, nq, pos0, kept, skip, t_hi, n_tiles, q_hi;   // key tiles (pages): the `kept` first ones, then from kept + skip to t_hi
   bool valid;           // false: past the end of a shorter sequence -- nothing to do
 };
 __device__ __forceinline__ bool ft_item(const FtArgs& p, int round, FtItem& it) {
@@ -79,12 +81,14 @@ __device__ __forceinline__ bool ft_item(const FtArgs& p, int round, FtItem& it) 
   it.g = it.h / (p.H / p.G);
   int q_lo = it.pos0 + it.r0;
   it.q_hi = it.pos0 + it.r0 + it.nq - 1;
-  int k_first = first_seen(q_lo, p.window);
-  it.t_lo = k_first / FT_BK;
+  const SeenKeys seen(q_lo, it.q_hi, p.window, p.keep);
+  it.kept = seen.kept;
+  it.skip = seen.skip;
   it.t_hi = it.q_hi / FT_BK;
-  it.n_tiles = it.t_hi - it.t_lo + 1;
+  it.n_tiles = seen.pages;
   return true;
 }
+__device__ __forceinline__ int ft_tile(const FtItem& it, int j) { return j < it.kept ? j : j + it.skip; }
 
 __device__ __forceinline__ float ft_ex2(float x) {
   float y;
@@ -101,6 +105,20 @@ __device__ __forceinline__ float ft_tanh(float x) {
 // capped score is handed on as (cap / scale) * tanh(s * scale / cap).
 __device__ __forceinline__ uint32_t ft_cap(uint32_t s, float cap_out, float cap_in) {
   return __float_as_uint(cap_out * ft_tanh(__uint_as_float(s) * cap_in));
+}
+// 32 output elements times the sigmoid of their gate logits (16-byte aligned)
+__device__ __forceinline__ void ft_gate(uint32_t (&v)[32], const bf16* g) {
+#pragma unroll
+  for (int c = 0; c < 4; c++) {
+    const uint4 w = *(const uint4*)(g + 8 * c);
+    const bf16* e = (const bf16*)&w;
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+      float s;
+      asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(s) : "f"(1.0f + ft_ex2(-FT_LOG2E * __bfloat162float(e[i]))));
+      v[8 * c + i] = __float_as_uint(__uint_as_float(v[8 * c + i]) * s);
+    }
+  }
 }
 __device__ __forceinline__ float ft_max3(float a, float b, float c) {
   float y;
@@ -201,7 +219,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         for (int j = 0; j < it.n_tiles; j++) {
           int s = J % FT_STAGES;
           if (!mbar_wait(b_kvempty + 8 * s, ((J / FT_STAGES) & 1) ^ 1, abort)) { ok = false; break; }
-          int page = bt[it.t_lo + j];
+          int page = bt[ft_tile(it, j)];
           int krow = (page * p.G + it.g) * FT_BK;
           mbar_expect_tx(b_kvfull + 8 * s, 2 * KV_BYTES);
 #pragma unroll
@@ -270,12 +288,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     bool ok = true;
     for (int round = 0; ok && ft_item(p, round, it); round++) {
     if (!it.valid) continue;
-    const int n_tiles = it.n_tiles, t_lo = it.t_lo, t_hi = it.t_hi, q_hi = it.q_hi, nq = it.nq, row0 = it.row0, r0 = it.r0, h = it.h;
+    const int n_tiles = it.n_tiles, t_hi = it.t_hi, q_hi = it.q_hi, nq = it.nq, row0 = it.row0, r0 = it.r0, h = it.h;
     const int qpos = it.pos0 + r0 + r, qfirst = first_seen(qpos, p.window);
     float m_ref = -INFINITY, l = 0.f;              // reference maximum (raw score units) and sum relative to it
     for (int j = 0; j < n_tiles && ok; j++) {
       const int Jg = J0 + j;
-      int a = Jg & 1, t = t_lo + j;
+      int a = Jg & 1, t = ft_tile(it, j);
       ok = mbar_wait(b_sfull + 8 * a, (Jg >> 1) & 1, abort);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -289,13 +307,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         for (int i = 0; i < 32; i++) { s0[i] = ft_cap(s0[i], cap_out, cap_in); s1[i] = ft_cap(s1[i], cap_out, cap_in); }
       }
       // ---- mask, row maximum (raw scores; four independent chains)
-      bool need_mask = (t * FT_BK + FT_BK - 1 > qpos) || t * FT_BK < qfirst;
+      bool need_mask = (t * FT_BK + FT_BK - 1 > qpos) || (t * FT_BK < qfirst && t * FT_BK + FT_BK > p.keep);
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < 32; i++) {
           int k0 = t * FT_BK + i, k1 = k0 + 32;
-          if (!(k0 <= qpos && k0 >= qfirst)) s0[i] = 0xff800000u;   // -inf
-          if (!(k1 <= qpos && k1 >= qfirst)) s1[i] = 0xff800000u;
+          if (!key_seen(k0, qpos, qfirst, p.keep)) s0[i] = 0xff800000u;   // -inf
+          if (!key_seen(k1, qpos, qfirst, p.keep)) s1[i] = 0xff800000u;
         }
       }
       float mxa = ft_max3(__uint_as_float(s0[0]), __uint_as_float(s0[1]), __uint_as_float(s0[2]));
@@ -392,6 +410,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         tmem_ld32(t_lane + 128 + c0, v);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (r < nq) {
+          if (p.gate != nullptr) ft_gate(v, p.gate + (size_t)(row0 + r0 + r) * p.gate_ld + (size_t)h * FT_HD + c0);
 #pragma unroll
           for (int c = 0; c < 4; c++) {
             uint4 w;
@@ -421,12 +440,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 
 // One query tile of a pair.
 struct FpTile {
-  int h, r0, nq, q_hi, t_lo, t_hi, n_tiles;
+  int h, r0, nq, q_hi, kept, t_lo, t_hi, n_tiles;   // key tiles: the `kept` first ones, then t_lo ... t_hi
   bool valid;           // false: past the end of the sequence -- nothing to do
 };
 // What a block works on in its r-th round.
 struct FpItem {
-  int b, g, row0, pos0, seq_end, T_lo, n_union;
+  int b, g, row0, pos0, seq_end, kept, skip, n_union;   // key tiles fetched: the `kept` first ones, then from kept + skip on
   FpTile sub[2];
   bool valid;
 };
@@ -437,10 +456,11 @@ __device__ __forceinline__ void fp_tile(const FtArgs& p, FpTile& s, int h, int q
   s.nq = min(FT_BQ, S - s.r0);
   int q_lo = pos0 + s.r0;
   s.q_hi = pos0 + s.r0 + s.nq - 1;
-  int k_first = first_seen(q_lo, p.window);
-  s.t_lo = k_first / FT_BK;
+  const SeenKeys seen(q_lo, s.q_hi, p.window, p.keep);
+  s.kept = seen.kept;
+  s.t_lo = seen.kept + seen.skip;
   s.t_hi = s.q_hi / FT_BK;
-  s.n_tiles = s.t_hi - s.t_lo + 1;
+  s.n_tiles = seen.pages;
 }
 __device__ __forceinline__ bool fp_item(const FtArgs& p, int round, FpItem& it) {
   int G = gridDim.x;
@@ -469,13 +489,20 @@ __device__ __forceinline__ bool fp_item(const FtArgs& p, int round, FpItem& it) 
   fp_tile(p, it.sub[0], h0, qt0, S, it.pos0);
   fp_tile(p, it.sub[1], h1, qt1, S, it.pos0);
   it.valid = it.sub[0].valid;                      // the second tile of a pair is never valid without the first
-  int lo = it.sub[0].t_lo, hi = it.sub[0].t_hi;
-  if (it.sub[1].valid) { lo = min(lo, it.sub[1].t_lo); hi = max(hi, it.sub[1].t_hi); }
-  it.T_lo = lo;
-  it.n_union = hi - lo + 1;                        // key tiles T_lo ... T_lo + n_union - 1; every one is in either tile's range
+  // The first tile's window starts no later than the second's, so what the first keeps or has in its window's first page
+  // on covers the front of what the second sees; the second may keep more pages, which then follow the first's directly.
+  it.kept = it.sub[0].kept;
+  it.skip = it.sub[0].t_lo - it.kept;
+  int hi = it.sub[0].t_hi;
+  if (it.sub[1].valid) hi = max(hi, it.sub[1].t_hi);
+  it.n_union = hi + 1 - it.skip;
   return true;
 }
-__device__ __forceinline__ bool fp_active(const FpTile& s, int t) { return s.valid && t >= s.t_lo && t <= s.t_hi; }
+__device__ __forceinline__ int fp_union_tile(const FpItem& it, int u) { return u < it.kept ? u : u + it.skip; }
+__device__ __forceinline__ bool fp_active(const FpTile& s, int t) { return s.valid && t <= s.t_hi && (t >= s.t_lo || t < s.kept); }
+// the place of tile t among those the query tile takes, and the tile at a place
+__device__ __forceinline__ int fp_place(const FpTile& s, int t) { return t < s.kept ? t : t - s.t_lo + s.kept; }
+__device__ __forceinline__ int fp_tile_at(const FpTile& s, int j) { return j < s.kept ? j : j - s.kept + s.t_lo; }
 
 // maximum of a row's 64 scores, four chains of three-input maxima
 __device__ __forceinline__ float ft_rowmax(const uint32_t (&s)[64]) {
@@ -491,13 +518,13 @@ __device__ __forceinline__ float ft_rowmax(const uint32_t (&s)[64]) {
   return fmaxf(ft_max3(m[0], m[1], m[2]), m[3]);
 }
 // scores of keys the query at qpos does not see become -inf (tile t holds keys 64 t ... 64 t + 63)
-__device__ __forceinline__ void ft_mask(uint32_t (&s)[64], int t, int qpos, int qfirst) {
-  bool need = (t * FT_BK + FT_BK - 1 > qpos) || t * FT_BK < qfirst;
+__device__ __forceinline__ void ft_mask(uint32_t (&s)[64], int t, int qpos, int qfirst, int keep) {
+  bool need = (t * FT_BK + FT_BK - 1 > qpos) || (t * FT_BK < qfirst && t * FT_BK + FT_BK > keep);
   if (need) {
 #pragma unroll
     for (int i = 0; i < 64; i++) {
       int k = t * FT_BK + i;
-      if (!(k <= qpos && k >= qfirst)) s[i] = 0xff800000u;   // -inf
+      if (!key_seen(k, qpos, qfirst, keep)) s[i] = 0xff800000u;   // -inf
     }
   }
 }
@@ -588,7 +615,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           for (int u = 0; u < it.n_union; u++) {
             int s = JU % FT_STAGES;
             if (!mbar_wait(b_kvempty + 8 * s, ((JU / FT_STAGES) & 1) ^ 1, abort)) { ok = false; break; }
-            int page = bt[it.T_lo + u];
+            int page = bt[fp_union_tile(it, u)];
             int krow = (page * p.G + it.g) * FT_BK;
             mbar_expect_tx(b_kvfull + 8 * s, 2 * KV_BYTES);
 #pragma unroll
@@ -620,10 +647,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           ok = mbar_wait(b_qfull, I & 1, abort);
           I++;
           auto issue_s = [&](int u) -> bool {
-            const int JUg = JU0 + u, s = JUg % FT_STAGES, t = it.T_lo + u;
+            const int JUg = JU0 + u, s = JUg % FT_STAGES, t = fp_union_tile(it, u);
             if (!mbar_wait(b_kvfull + 8 * s, (JUg / FT_STAGES) & 1, abort)) return false;
             if (fp_active(sub, t)) {
-              const int Jg = J0 + t - sub.t_lo, sb = Jg % NBUF;
+              const int Jg = J0 + fp_place(sub, t), sb = Jg % NBUF;
               // S(Jg) takes the place of S(Jg - NBUF), which the softmax threads have taken into their registers: with
               // two buffers their P(Jg - 2) was waited for; the single buffer has a barrier for it
               if (NBUF == 1 && !mbar_wait(b_sub + SUB_BARS * x + B_SEMPTY + 8 * sb, ((Jg / NBUF) & 1) ^ 1, abort)) return false;
@@ -640,9 +667,9 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           if (ok) ok = issue_s(0);
           for (int u = 0; u < n_union && ok; u++) {
             if (u + 1 < n_union) { ok = issue_s(u + 1); if (!ok) break; }
-            const int JUg = JU0 + u, s = JUg % FT_STAGES, t = it.T_lo + u;
+            const int JUg = JU0 + u, s = JUg % FT_STAGES, t = fp_union_tile(it, u);
             if (fp_active(sub, t)) {
-              const int j = t - sub.t_lo, Jg = J0 + j, a = Jg & 1;
+              const int j = fp_place(sub, t), Jg = J0 + j, a = Jg & 1;
               ok = mbar_wait(b_sub + SUB_BARS * x + B_PFULL + 8 * a, (Jg >> 1) & 1, abort);   // P of this tile is written, and O has been rescaled if it had to be
               if (!ok) break;
               asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -673,9 +700,9 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     for (int round = 0; ok && fp_item(p, round, it); round++) {
     if (!it.valid) continue;
     const FpTile sb = it.sub[x];
-    const int n_union = it.n_union, T_lo = it.T_lo;
+    const int n_union = it.n_union;
     if (sb.valid) {
-    const int n_tiles = sb.n_tiles, t_lo = sb.t_lo, seq_end = it.seq_end;
+    const int n_tiles = sb.n_tiles, seq_end = it.seq_end;
     const int qpos = it.pos0 + sb.r0 + r, qfirst = first_seen(qpos, p.window);
     float m_ref = -INFINITY, l = 0.f;              // reference maximum (raw score units) and sum relative to it
     uint32_t s[64];
@@ -683,7 +710,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll 1
     for (int j = 0; j < n_tiles && ok; j++) {
       const int Jg = J0 + j;
-      const int a = Jg & 1, t = t_lo + j, bf = Jg % NBUF;
+      const int a = Jg & 1, t = fp_tile_at(sb, j), bf = Jg % NBUF;
       ok = mbar_wait(b_sfull + 8 * bf, (Jg / NBUF) & 1, abort);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -699,7 +726,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int i = 0; i < 64; i++) s[i] = ft_cap(s[i], cap_out, cap_in);
       }
-      ft_mask(s, t, qpos, qfirst);
+      ft_mask(s, t, qpos, qfirst, p.keep);
       mx = ft_rowmax(s);
       // ---- move the reference maximum only when the row's maximum has outgrown it by 2^8
       bool grow = mx > m_ref && (m_ref == -INFINITY || (mx - m_ref) * sc > 8.0f);
@@ -749,7 +776,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // keys of the sequence's last page beyond its last position hold whatever the page held before:
         // their probabilities are zero, but 0 * NaN is NaN, so their value rows are cleared -- by either
         // tile of the pair that takes this page, each before its own P V product (zeros over zeros harm nothing)
-        const int JUg = JU0 + t - T_lo, st = JUg % FT_STAGES, n_valid = max(0, seq_end + 1 - t * FT_BK);
+        const int JUg = JU0 + (t < it.kept ? t : t - it.skip), st = JUg % FT_STAGES, n_valid = max(0, seq_end + 1 - t * FT_BK);
         ok = mbar_wait(b_kvfull + 8 * st, (JUg / FT_STAGES) & 1, abort);
         if (!ok) break;
         for (int e = q * 32 + lane; e < (FT_BK - n_valid) * 8 * NA; e += 128) {
@@ -779,6 +806,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         tmem_ld32(t_lane + 128 + c0, v);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (r < sb.nq) {
+          if (p.gate != nullptr) ft_gate(v, p.gate + (size_t)(it.row0 + sb.r0 + r) * p.gate_ld + (size_t)sb.h * FT_HD + c0);
 #pragma unroll
           for (int c = 0; c < 4; c++) {
             uint4 w;
@@ -845,11 +873,13 @@ static int fp_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 // [n_pages][G][64][hd] with n_pages the number of pages the storage holds; hd 64 or 128.
 SLLM_EXPORT int sllm_attn_prefill_tc_bf16(const void* q, int q_ld, int T, void* out, const int* seq_start, const int* seq_pos0,
                                           const int* block_table, int max_pages, const void* kpages, const void* vpages,
-                                          long long n_pages, int B, int max_new, int H, int G, int hd, int window, float scale,
-                                          float softcap, const float* sink, int* err, cudaStream_t stream) {
+                                          long long n_pages, int B, int max_new, int H, int G, int hd, int window, int keep, float scale,
+                                          float softcap, const float* sink, const void* gate, int gate_ld, int* err,
+                                          cudaStream_t stream) {
   if (B <= 0 || max_new <= 0) return 0;
   if ((hd != 64 && hd != 128) || G < 1 || H % G != 0 || (q_ld & 7) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
-      ((uintptr_t)kpages & 15) || ((uintptr_t)vpages & 15))
+      ((uintptr_t)kpages & 15) || ((uintptr_t)vpages & 15) || keep < 0 ||
+      (gate && (((uintptr_t)gate & 15) || (gate_ld & 7) || gate_ld < H * hd)))
     return SLLM_ERR_ARG;
   long long kv_rows = n_pages * G * FT_BK;
   if (kv_rows <= 0 || kv_rows > 0x7fffffffLL) return SLLM_ERR_ARG;
@@ -871,13 +901,15 @@ SLLM_EXPORT int sllm_attn_prefill_tc_bf16(const void* q, int q_ld, int T, void* 
     if (e != cudaSuccess) return (int)e;
   }
   if (hd == 64) {
-    FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, window, scale, err, n_qt, B, (int)n_items, 0, softcap, sink};
+    FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, window, keep, scale, err, n_qt, B, (int)n_items, 0, softcap, sink,
+             (const bf16*)gate, gate_ld};
     dim3 grid((unsigned)(n_items < 2LL * sm_count ? n_items : 2LL * sm_count));     // two blocks per SM that stay
     return ft_launch<64, 3>(mq, mk, mv, a, grid, stream);
   }
   int pair_heads = ((H / G) % 2 == 0) ? 1 : 0;
   n_items = pair_heads ? (long long)(H / 2) * n_qt * B : (long long)H * ((n_qt + 1) / 2) * B;
-  FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, window, scale, err, n_qt, B, (int)n_items, pair_heads, softcap, sink};
+  FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, window, keep, scale, err, n_qt, B, (int)n_items, pair_heads, softcap, sink,
+           (const bf16*)gate, gate_ld};
   dim3 grid((unsigned)(n_items < (long long)sm_count ? n_items : (long long)sm_count));       // one block per SM that stays
   return fp_launch<128, 4>(mq, mk, mv, a, grid, stream);
 }

@@ -109,6 +109,19 @@ class KernelSet:
                                            _ptr(last, torch.int32, "last"), _ptr(err_flag, torch.int32, "err"), _stream()),
                "embed_pair_rows")
 
+    def embed_rows_sinusoid(self, ids, tok_pos, table, coarse, fine, out, err_flag):
+        """out float32 [T, d] = table[ids[t]] plus sine (even columns) and cosine (odd ones) of the position's angles;
+        coarse float32 [n, pairs, 2], fine float32 [64, pairs, 2]: (sin, cos) of positions 64 a and b."""
+        T, d = out.shape
+        pairs = (d + 1) // 2
+        if tuple(coarse.shape[1:]) != (pairs, 2) or tuple(fine.shape) != (64, pairs, 2) or table.shape[1] != d:
+            raise KernelError(f"embed_rows_sinusoid: tables {tuple(coarse.shape)}, {tuple(fine.shape)} for rows of {d}")
+        _check(self._fn("embed_rows_sinusoid")(_ptr(ids, torch.int32, "ids"), _ptr(tok_pos, torch.int32, "tok_pos"),
+                                               _ptr(table, self.dtype, "table"), _ptr(coarse, torch.float32, "coarse"),
+                                               _ptr(fine, torch.float32, "fine"), _ptr(out, torch.float32, "out"), c_int(T), c_int(d),
+                                               c_int(table.shape[0]), c_int(coarse.shape[0]), _ptr(err_flag, torch.int32, "err"),
+                                               _stream()), "embed_rows_sinusoid")
+
     # ------------------------------------------------------------------ norm
     def add_rmsnorm(self, x, delta, rows, weight, y, eps):
         """x float32 [T,d] residual (+= delta when rows is None); y [n,d] normed output. delta: None,
@@ -173,23 +186,25 @@ class KernelSet:
 
     # ------------------------------------------------------------------ attention
     def attn_paged(self, q, out, seq_start, seq_pos0, block_table, kpages, vpages, n_seqs, max_new, n_heads, n_kv,
-                   head_dim, window, scale, softcap=None, sink=None):
+                   head_dim, window, scale, softcap=None, sink=None, v_dim=None, keep=0):
         """`softcap`: a score s becomes softcap * tanh(s / softcap) before the softmax; `sink` float32 [n_heads]:
-        exp(sink[h]) joins head h's denominator with no key and no value."""
+        exp(sink[h]) joins head h's denominator with no key and no value. `v_dim`: the values' width where it is not
+        the keys'; `keep`: the first positions of a sequence that stay visible behind the window."""
         _check(self._fn("attn_paged")(_ptr(q, self.dtype, "q"), c_int(q.shape[1]), _ptr(out, self.dtype, "out"),
                                       _ptr(seq_start, torch.int32, "seq_start"), _ptr(seq_pos0, torch.int32, "seq_pos0"),
                                       _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]),
                                       _ptr(kpages, self.dtype, "kpages"), _ptr(vpages, self.dtype, "vpages"),
                                       c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv), c_int(head_dim),
-                                      c_int(window or 0), c_float(scale), c_float(softcap or 0.0),
-                                      _ptr(sink, torch.float32, "sink"), _stream()), "attn_paged")
+                                      c_int(v_dim or head_dim), c_int(window or 0), c_int(keep), c_float(scale),
+                                      c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), _stream()), "attn_paged")
 
     def attn_decode_split(self, q, out, seq_pos0, block_table, kpages, vpages, part, n_seqs, n_heads, n_kv, head_dim,
-                          window, scale, n_split, softcap=None, sink=None):
+                          window, scale, n_split, softcap=None, sink=None, v_dim=None, keep=0):
         """One query per sequence, each sequence's keys split over `n_split` blocks (then merged);
-        `part`: float32 scratch of n_seqs * n_heads * n_split * (head_dim + 2) elements, or None for one split.
-        `softcap`, `sink`: as for `attn_paged`; the sink joins once, where the splits are merged."""
-        need = n_seqs * n_heads * n_split * (head_dim + 2) if n_split > 1 else 0
+        `part`: float32 scratch of n_seqs * n_heads * n_split * (v_dim + 2) elements, or None for one split.
+        `softcap`, `sink`, `v_dim`, `keep`: as for `attn_paged`; the sink joins once, where the splits are merged."""
+        v_dim = v_dim or head_dim
+        need = n_seqs * n_heads * n_split * (v_dim + 2) if n_split > 1 else 0
         if need and (part is None or part.numel() < need):
             raise KernelError(f"attn_decode_split scratch holds {0 if part is None else part.numel()} floats, needs {need}")
         _check(self._fn("attn_decode_split")(_ptr(q, self.dtype, "q") if q.is_contiguous() else c_void_p(q.data_ptr()),
@@ -198,13 +213,13 @@ class KernelSet:
                                              _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]),
                                              _ptr(kpages, self.dtype, "kpages"), _ptr(vpages, self.dtype, "vpages"),
                                              _ptr(part, torch.float32, "part"), c_int(n_seqs), c_int(n_heads), c_int(n_kv),
-                                             c_int(head_dim), c_int(window or 0), c_float(scale), c_int(n_split),
-                                             c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), _stream()),
+                                             c_int(head_dim), c_int(v_dim), c_int(window or 0), c_int(keep), c_float(scale),
+                                             c_int(n_split), c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), _stream()),
                "attn_decode_split")
 
     @staticmethod
-    def attn_decode_split_takes(head_dim: int, q_ld: int) -> bool:
-        return head_dim % 4 == 0 and 4 <= head_dim <= 512 and q_ld % 4 == 0
+    def attn_decode_split_takes(head_dim: int, q_ld: int, v_dim: int | None = None) -> bool:
+        return all(w % 4 == 0 and 4 <= w <= 512 for w in (head_dim, v_dim or head_dim)) and q_ld % 4 == 0
 
     @staticmethod
     def attn_decode_splits(n_seqs: int, n_heads: int, n_kv: int, pages: int, sm_count: int) -> int:
@@ -461,24 +476,45 @@ class PrefillAttentionTC:
         self.lib.sllm_attn_prefill_tc_bf16.restype = c_int
 
     def attn(self, q, out, seq_start, seq_pos0, block_table, kpages, vpages, n_seqs, max_new, n_heads, n_kv, head_dim,
-             window, scale, err_flag, softcap=None, sink=None):
+             window, scale, err_flag, softcap=None, sink=None, keep=0, gate=None):
         """`softcap`: a score s becomes softcap * tanh(s / softcap) before the softmax; `sink` float32 [n_heads]: exp(sink[h])
-        joins head h's denominator with no key and no value."""
+        joins head h's denominator with no key and no value; `keep`: the first positions of a sequence that stay visible behind
+        the window; `gate`: bfloat16 [T, n_heads * head_dim] (a column slice), whose sigmoid multiplies the output."""
+        gp, gl = _gate_args(gate, q.shape[0], n_heads * head_dim)
         _check(self.lib.sllm_attn_prefill_tc_bf16(
             _ptr(q, torch.bfloat16, "q"), c_int(q.shape[1]), c_int(q.shape[0]), _ptr(out, torch.bfloat16, "out"),
             _ptr(seq_start, torch.int32, "seq_start"), _ptr(seq_pos0, torch.int32, "seq_pos0"),
             _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]),
             _ptr(kpages, torch.bfloat16, "kpages"), _ptr(vpages, torch.bfloat16, "vpages"), c_longlong(kpages.shape[0]),
-            c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(window or 0), c_float(scale),
-            c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), _ptr(err_flag, torch.int32, "err_flag"), _stream()),
-            "attn_prefill_tc")
+            c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(window or 0), c_int(keep),
+            c_float(scale), c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), gp, gl, _ptr(err_flag, torch.int32, "err_flag"),
+            _stream()), "attn_prefill_tc")
+
+
+def _gate_args(gate, rows: int, cols: int):
+    """Pointer and row stride of bfloat16 gate logits [rows, cols], a column slice of a wider buffer; (null, 0) without."""
+    if gate is None:
+        return c_void_p(0), c_int(0)
+    if not gate.is_cuda or gate.dtype != torch.bfloat16 or tuple(gate.shape) != (rows, cols) or gate.stride(1) != 1:
+        raise KernelError(f"gate logits {tuple(gate.shape)} {gate.dtype} for an output of {(rows, cols)}")
+    return c_void_p(gate.data_ptr()), c_int(gate.stride(0))
+
+
+def gate_aligned(gate) -> bool:
+    """Whether attention kernels can read these gate logits with 16-byte accesses."""
+    return gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0
 
 
 class PrefillAttentionMMA:
     """Causal attention of a prompt step on mma.sync for key and value widths the tcgen05 kernels do not take (bfloat16): keys
-    of 64, 96, 128, 192 or 256, values of 64 or 128; rows in storage may be wider than what is used."""
+    up to 256, values up to 128, in multiples of 8 (built for the widths below; what is missing is zeros on the chip); rows
+    in storage may be wider than what is used."""
     KEY_WIDTHS = (64, 96, 128, 192, 256)
     VALUE_WIDTHS = (64, 128)
+
+    @staticmethod
+    def takes(key_dim: int, value_dim: int) -> bool:
+        return key_dim % 8 == 0 and 8 <= key_dim <= 256 and value_dim % 8 == 0 and 8 <= value_dim <= 128
 
     def __init__(self):
         self.lib = load_library("attn_prefill_mma")
@@ -492,16 +528,18 @@ class PrefillAttentionMMA:
         return None if k is None or v is None else (k, v)
 
     def attn(self, q, q_hw, out, o_hw, seq_start, seq_pos0, block_table, kpages, vpages, n_seqs, max_new, n_heads, n_kv, kd, vd,
-             window, scale, softcap=None, sink=None):
+             window, scale, softcap=None, sink=None, keep=0, gate=None):
         """q [T, n_heads * q_hw], out [T, n_heads * o_hw] (the o_hw - vd columns past a head's values are set to 0), kpages
-        [pages, n_kv, 64, k_w], vpages [pages, n_kv, 64, v_w]; kd and vd are the widths used."""
+        [pages, n_kv, 64, k_w], vpages [pages, n_kv, 64, v_w]; kd and vd are the widths used. `keep`, `gate` (bfloat16
+        [T, n_heads * vd]): as for `PrefillAttentionTC.attn`."""
+        gp, gl = _gate_args(gate, q.shape[0], n_heads * vd)
         _check(self.lib.sllm_attn_prefill_mma_bf16(
             _ptr(q, torch.bfloat16, "q"), c_int(q.shape[1]), c_int(q_hw), _ptr(out, torch.bfloat16, "out"), c_int(out.shape[1]),
             c_int(o_hw), _ptr(seq_start, torch.int32, "seq_start"), _ptr(seq_pos0, torch.int32, "seq_pos0"),
             _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]), _ptr(kpages, torch.bfloat16, "kpages"),
             c_int(kpages.shape[-1]), _ptr(vpages, torch.bfloat16, "vpages"), c_int(vpages.shape[-1]), c_int(n_seqs), c_int(max_new),
-            c_int(n_heads), c_int(n_kv), c_int(kd), c_int(vd), c_int(window or 0), c_float(scale), c_float(softcap or 0.0),
-            _ptr(sink, torch.float32, "sink"), _stream()), "attn_prefill_mma")
+            c_int(n_heads), c_int(n_kv), c_int(kd), c_int(vd), c_int(window or 0), c_int(keep), c_float(scale), c_float(softcap or 0.0),
+            _ptr(sink, torch.float32, "sink"), gp, gl, _stream()), "attn_prefill_mma")
 
 
 class DecodeKernels:
@@ -512,7 +550,8 @@ class DecodeKernels:
     def __init__(self):
         self.lib = load_library("decode_bf16")
         for n in ("sllm_gemm_small_m_bf16", "sllm_gemm_small_m_fold_bf16", "sllm_attn_decode_bf16",
-                  "sllm_attn_decode_merged_bf16", "sllm_attn_decode_rope_bf16", "sllm_attn_decode_capped_bf16"):
+                  "sllm_attn_decode_merged_bf16", "sllm_attn_decode_rope_bf16", "sllm_attn_decode_capped_bf16",
+                  "sllm_attn_decode_general_bf16"):
             getattr(self.lib, n).restype = c_int
         self.lib.sllm_attn_decode_scratch_bytes.restype = c_longlong
         self.lib.sllm_attn_decode_uses_mma.restype = c_int
@@ -682,6 +721,34 @@ class DecodeKernels:
             _ptr(vpages, torch.bfloat16, "vpages"), _ptr(scratch, torch.float32, "scratch"), _ptr(tickets, torch.int32, "tickets"),
             c_int(n_seqs), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(window or 0), c_float(scale), c_int(n_split),
             c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), _stream()), "attn_decode_capped")
+
+    @staticmethod
+    def general_takes(head_dim: int, v_dim: int) -> bool:
+        return head_dim % 8 == 0 and 8 <= head_dim <= 256 and v_dim % 8 == 0 and 8 <= v_dim <= 128
+
+    @staticmethod
+    def general_splits(n_seqs: int, n_kv_heads: int, head_dim: int, v_dim: int, pages: int, sm_count: int) -> int:
+        """Over how many blocks `attn_decode_general` splits each sequence's keys: as `attention_splits` for its kernel, but
+        down to two pages a block (a window has few)."""
+        want = ((4 if max(head_dim, v_dim) <= 64 else 2) * sm_count) // max(1, n_seqs * n_kv_heads)
+        n = max(1, min(want, pages // 2, DecodeKernels.MAX_SPLITS))
+        per = -(-pages // n)
+        return max(1, -(-pages // per))
+
+    def attn_decode_general(self, q, out, seq_pos0, block_table, kpages, vpages, scratch, tickets, n_seqs, n_heads, n_kv, head_dim,
+                            v_dim, window, scale, n_split, keep=0, softcap=None, sink=None, gate=None):
+        """Decode attention on the tensor-core kernel for keys head_dim and values v_dim wide (multiples of 8 up to 256 and
+        128), with the first `keep` positions visible behind any window, capped scores, a sink per head (float32 [n_heads])
+        and a gate (bfloat16 [n_seqs, n_heads * v_dim]) on the output; scratch: n_seqs * n_heads * n_split * (v_dim + 2) floats."""
+        if scratch.numel() < n_seqs * n_heads * n_split * (v_dim + 2) or tickets.numel() < n_seqs * n_kv:
+            raise KernelError("attn_decode_general: scratch or tickets too small")
+        gp, gl = _gate_args(gate, n_seqs, n_heads * v_dim)
+        _check(self.lib.sllm_attn_decode_general_bf16(
+            _ptr(q, torch.bfloat16, "q"), c_int(q.shape[1]), _ptr(out, torch.bfloat16, "out"), _ptr(seq_pos0, torch.int32, "seq_pos0"),
+            _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]), _ptr(kpages, torch.bfloat16, "kpages"),
+            _ptr(vpages, torch.bfloat16, "vpages"), _ptr(scratch, torch.float32, "scratch"), _ptr(tickets, torch.int32, "tickets"),
+            c_int(n_seqs), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(v_dim), c_int(window or 0), c_int(keep), c_float(scale),
+            c_int(n_split), c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), gp, gl, _stream()), "attn_decode_general")
 
 
 class SequenceKernels:
@@ -1060,23 +1127,37 @@ class GateKernels:
     _view = staticmethod(SequenceKernels._view)
 
     def qk_norm_store(self, c, q_out, tok_pos, tok_seq, block_table, cos_sin, kpages, vpages, n_heads, n_kv, head_dim, v_dim,
-                      rot, interleaved, q_weight, k_weight, eps):
-        """Row t of c (float32 or element type; a view) holds [queries | keys | values] of a token. Queries and keys are
-        each divided by the root mean square of their whole part and multiplied by q_weight / k_weight (None: as
+                      rot, interleaved, q_weight, k_weight, eps, bias=None, per_head=False, value_mix=None):
+        """Row t of c (float32 or element type; a view) holds [queries | keys | values] of a token; `bias` (float32, the
+        same columns) is added first. Queries and keys are each divided by the root mean square of their whole part
+        (`per_head`: of every head by itself, weights of one head's width) and multiplied by q_weight / k_weight (None: as
         they are), turned by the table over their first `rot` dims, and go to q_out [T, n_heads * head_dim] and, with
-        the values, to the rows' places in the cache pages (n_kv == 0: queries only)."""
+        the values, to the rows' places in the cache pages (n_kv == 0: queries only). `value_mix` = (kept, None): the values
+        also go to kept [T, n_kv * v_dim] (element type); (kept, lam): stored are (1 - lam) * values + lam * kept."""
+        if bias is not None and bias.numel() != (n_heads + n_kv) * head_dim + n_kv * v_dim:
+            raise KernelError(f"qk_norm_store: a bias of {bias.numel()} columns")
+        for w, heads in ((q_weight, n_heads), (k_weight, n_kv)):
+            if w is not None and w.numel() != (head_dim if per_head else heads * head_dim):
+                raise KernelError(f"qk_norm_store: a norm weight of {w.numel()} for {heads} heads of {head_dim}")
+        kept, lam, mode = None, 0.0, 0
+        if value_mix is not None:
+            kept, mode = value_mix[0], 1 if value_mix[1] is None else 2
+            lam = value_mix[1] or 0.0
+            if tuple(kept.shape) != (c.shape[0], n_kv * v_dim):
+                raise KernelError(f"qk_norm_store: kept values {tuple(kept.shape)} for {n_kv} heads of {v_dim}")
         w_f32 = 0
         for w in (q_weight, k_weight):
             if w is not None:
                 w_f32 = self._flag(w, "norm weight")
         _check(self._fn("qk_norm_store")(
-            self._view(c, "c"), c_int(self._flag(c, "c")), c_int(c.stride(0)), self._view(q_out, "q_out"), c_int(q_out.stride(0)),
-            _ptr(tok_pos, torch.int32, "tok_pos"), _ptr(tok_seq, torch.int32, "tok_seq"),
+            self._view(c, "c"), c_int(self._flag(c, "c")), c_int(c.stride(0)), _ptr(bias, torch.float32, "bias"),
+            self._view(q_out, "q_out"), c_int(q_out.stride(0)), _ptr(tok_pos, torch.int32, "tok_pos"), _ptr(tok_seq, torch.int32, "tok_seq"),
             _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1] if block_table is not None else 0),
             _ptr(cos_sin, torch.float32, "cos_sin"), _ptr(kpages, self.dtype if kpages is not None else None, "kpages"),
             _ptr(vpages, self.dtype if vpages is not None else None, "vpages"), c_int(c.shape[0]), c_int(n_heads), c_int(n_kv),
             c_int(head_dim), c_int(v_dim), c_int(rot), c_int(1 if interleaved else 0), _ptr(q_weight, None, "q_weight"),
-            _ptr(k_weight, None, "k_weight"), c_int(w_f32), c_float(eps), _stream()), "qk_norm_store")
+            _ptr(k_weight, None, "k_weight"), c_int(w_f32), c_int(1 if per_head else 0), c_float(eps),
+            _ptr(kept, self.dtype if kept is not None else None, "kept"), c_int(mode), c_float(lam), _stream()), "qk_norm_store")
 
     FUSED_CONV_MAX_WIDTH = 200 * 1024 // 4      # the row stays in shared memory as floats
 
@@ -1146,8 +1227,9 @@ class GateKernels:
                                          _ptr(out, self.dtype, "out"), c_int(a.shape[0]), c_int(a.shape[1]), _stream()),
                "gelu_mul_rows")
 
-    def add_rms_normed(self, x, y, weight, eps, norm=None, rows=None, vec=None, dyt=None):
-        """x float32 [T, d] += y / sqrt(mean(y^2) + eps) * weight; y [T, d] or [P, T, d] partial sums (float32 or element type).
+    def add_rms_normed(self, x, y, weight, eps, norm=None, rows=None, vec=None, dyt=None, y_bias=None, copy=None):
+        """x float32 [T, d] += y / sqrt(mean(y^2) + eps) * weight; y [T, d] or [P, T, d] partial sums (float32 or element type),
+        to which `y_bias` (float32 [d]) is added first. `copy` (element type [T, d]) receives the stream as it then stands.
         `norm` = (weight2, eps2, out): in the same pass out (element type) = x / sqrt(mean(x^2) + eps2) * weight2 of the
         stream as it then stands; with `rows` (int32 on the device) only those rows are worked on and out has a row for each.
         `dyt` = (weight2, bias2, alpha2, out), all float32: the norm that follows is tanh(alpha2 x) * weight2 + bias2 instead.
@@ -1161,17 +1243,24 @@ class GateKernels:
             norm = (w2, 0.0, out)
             if w2.dtype != torch.float32 or b2.dtype != torch.float32 or b2.shape[0] != x.shape[1]:
                 raise KernelError("the norm without statistics takes float32 weight and bias of the stream's width")
+        if copy is not None:
+            if norm is not None or rows is not None:
+                raise KernelError("a copy of the stream is written where no norm follows the sum")
+            norm = (None, 0.0, copy)
+        if y_bias is not None and y_bias.numel() != x.shape[1]:
+            raise KernelError(f"a bias of {y_bias.numel()} for rows of {x.shape[1]}")
         if tuple(y.shape[-2:]) != tuple(x.shape) or not y.is_contiguous() or (rows is not None and norm is None):
             raise KernelError(f"y {tuple(y.shape)} does not fit the stream {tuple(x.shape)}")
         if vec is not None and (vec.dtype != torch.float32 or vec.numel() != x.shape[1]):
             raise KernelError(f"the row vector {tuple(vec.shape)} {vec.dtype} does not fit the stream {tuple(x.shape)}")
         w2, eps2, out = norm if norm is not None else (None, 0.0, None)
         n_out = 0 if norm is None else (x.shape[0] if rows is None else rows.shape[0])
-        if norm is not None and (tuple(out.shape) != (n_out, x.shape[1]) or not out.is_contiguous() or w2.shape[0] != x.shape[1]):
+        if norm is not None and (tuple(out.shape) != (n_out, x.shape[1]) or not out.is_contiguous()
+                                 or (w2 is not None and w2.shape[0] != x.shape[1])):
             raise KernelError(f"the norm's output {tuple(out.shape)} does not fit {n_out} rows of the stream {tuple(x.shape)}")
         _check(self._fn("add_rms_normed")(_ptr(x, torch.float32, "x"), _ptr(y, None, "y"), c_int(self._flag(y, "y")), c_int(P),
-                                          c_int(x.shape[0]), _ptr(weight, None, "weight"), c_int(self._flag(weight, "weight")),
-                                          c_int(x.shape[1]), c_float(eps), _ptr(rows, torch.int32, "rows"), c_int(n_out),
+                                          c_int(x.shape[0]), _ptr(y_bias, torch.float32, "y_bias"),
+                                          _ptr(weight, None, "weight"), c_int(self._flag(weight, "weight")), c_int(x.shape[1]), c_float(eps), _ptr(rows, torch.int32, "rows"), c_int(n_out),
                                           _ptr(w2, None, "weight2"), c_int(self._flag(w2, "weight2") if w2 is not None else 0),
                                           c_float(eps2), _ptr(out, self.dtype if out is not None else None, "out"),
                                           _ptr(vec, torch.float32, "vec"), _ptr(b2, torch.float32, "bias2"), c_float(alpha2), _stream()),

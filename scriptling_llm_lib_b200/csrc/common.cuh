@@ -29,11 +29,33 @@ __host__ __device__ __forceinline__ int first_seen(int qpos, int window) {
   return window < 0 ? qpos - qpos % (-window) : 0;
 }
 
+// The keys that consecutive queries q_lo .. q_hi see between them when, beside `window`, the first `keep` positions of the
+// sequence stay visible to every later query: whole pages, the kept ones first, then those from the window's first page
+// on. The pages between the two are skipped; they may have gone back to the pool. A walk goes over dense page numbers
+// 0 .. pages - 1 (or dense key numbers); `page(v)` and `key(x)` give the place in the sequence. keep == 0: the window alone.
+struct SeenKeys {
+  int kept, skip, pages;   // pages kept at the front, pages left out behind them, pages to walk
+  __host__ __device__ __forceinline__ SeenKeys(int q_lo, int q_hi, int window, int keep) {
+    int first_page = first_seen(q_lo, window) / SLLM_PAGE, kp = (keep + SLLM_PAGE - 1) / SLLM_PAGE;
+    kept = kp < first_page ? kp : first_page;
+    skip = first_page - kept;
+    pages = q_hi / SLLM_PAGE + 1 - skip;
+  }
+  __host__ __device__ __forceinline__ int page(int v) const { return v < kept ? v : v + skip; }
+  __host__ __device__ __forceinline__ int key(int x) const { return x < kept * SLLM_PAGE ? x : x + skip * SLLM_PAGE; }
+};
+// whether a query at `qpos`, whose window starts at `first`, sees key `k`
+__host__ __device__ __forceinline__ bool key_seen(int k, int qpos, int first, int keep) {
+  return k <= qpos && (k >= first || k < keep);
+}
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(bf16 v) { return __bfloat162float(v); }
 template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float sigmoid_of(float v) { return 1.0f / (1.0f + expf(-v)); }
 
 // weights of a norm may be stored in bfloat16 or float32 whatever the activation type
 __device__ __forceinline__ float load_w(const void* w, int is_f32, int j) {

@@ -370,7 +370,18 @@ struct AttnDecodeArgs {
   // null) [H]: exp(sink[h]) joins head h's denominator once, where the splits are merged (no key, no value)
   float softcap;
   const float* sink;
+  // the tensor-core kernel only: key and value widths of its trimmed form (else both HD); the first `keep` positions stay
+  // visible behind any window; gate (or null) [B, gate_ld]: output element (h, d) is multiplied by the sigmoid of column h * vd + d
+  int hd, vd, keep;
+  const bf16* gate;
+  int gate_ld;
 };
+
+// a finished output element times its gate
+__device__ __forceinline__ bf16 ad_gated(const AttnDecodeArgs& p, float v, int b, int col) {
+  if (p.gate != nullptr) v *= sigmoid_of(to_f32(ld_dep(p.gate + (size_t)b * p.gate_ld + col)));
+  return __float2bfloat16_rn(v);
+}
 
 // the softmax denominator ls (relative to the maximum mn, base 2) once a sink has joined it
 __device__ __forceinline__ float ad_sink_joined(float ls, float mn, const float* sink, int h) {
@@ -468,7 +479,7 @@ __device__ __forceinline__ void ad_ticket_merge(const AttnDecodeArgs& p, int b, 
 #pragma unroll 8
         for (int s2 = 0; s2 < p.n_split; s2++) a += __ldcg(src + (size_t)s2 * (HD + 2)) * sm_c[r][s2];
         float ls = sm_l[r];
-        p.out[((size_t)b * p.H + h) * HD + dd] = __float2bfloat16_rn(ls > 0.f ? a / ls : 0.f);
+        p.out[((size_t)b * p.H + h) * HD + dd] = ad_gated(p, ls > 0.f ? a / ls : 0.f, b, h * HD + dd);
       }
       __syncthreads();
     }
@@ -488,7 +499,7 @@ __device__ __forceinline__ void ad_ticket_merge(const AttnDecodeArgs& p, int b, 
       ls += __ldcg(ps + HD + 1) * c;
     }
     ls = ad_sink_joined(ls, mn, p.sink, h);
-    p.out[((size_t)b * p.H + h) * HD + dd] = __float2bfloat16_rn(ls > 0.f ? a / ls : 0.f);
+    p.out[((size_t)b * p.H + h) * HD + dd] = ad_gated(p, ls > 0.f ? a / ls : 0.f, b, h * HD + dd);
   }
 }
 
@@ -739,14 +750,18 @@ __global__ void __launch_bounds__(AD_WARPS * 32, NREP == 1 ? 7 : 1) attn_decode_
 //     output tile jt is dim n*8 + jt.
 // UP: rows 8..15 carry heads too (more than 8 heads per group). The maximum is kept per row over
 // the four lanes that share it, and the running output is rescaled only when some row's grew.
-template <int HD, bool UP, bool RAW>
+// Keys are KD wide and values VD wide. TRIM: they are p.hd <= KD and p.vd <= VD, multiples of 8 (what is missing is zeros
+// in the fragments); else both are what the kernel is built for. The walk goes over dense page numbers (SeenKeys).
+template <int KD, int VD, bool UP, bool RAW, bool TRIM>
 __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDecodeArgs p) {
+  static_assert(!RAW || (KD == VD && !TRIM), "raw rows: keys and values of one width");
   constexpr int ROWS = UP ? 16 : 8;
-  constexpr int CH = HD / 8;       // 16-byte chunks of a head row
-  constexpr int NJ = HD / 32;      // pairs of k-steps of the score product
-  constexpr int NC = HD / 64;      // 64-dim column blocks of the output
-  __shared__ __align__(16) bf16 sm_q[ROWS][HD];
-  __shared__ float sm_acc[AD_WARPS][ROWS][HD + 1];
+  constexpr int CH = KD / 8;       // 16-byte chunks of a query or key row
+  constexpr int NJ = KD / 32;      // pairs of k-steps of the score product
+  constexpr int NC = VD / 64;      // 64-dim column blocks of the output
+  const int hd = TRIM ? p.hd : KD, vd = TRIM ? p.vd : VD;
+  __shared__ __align__(16) bf16 sm_q[ROWS][KD];
+  __shared__ float sm_acc[AD_WARPS][ROWS][VD + 1];
   __shared__ float sm_ml[AD_WARPS][ROWS][2];
   pdl_launch_dependents();
   if (!RAW) pdl_wait();        // given finished queries, the kernel in front may have written any of its inputs
@@ -754,10 +769,14 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = lane >> 2, t = lane & 3;
   const int pos = p.seq_pos0[b];
   const int k_begin = first_seen(pos, p.window);
-  const int pb = k_begin / SLLM_PAGE, pe = pos / SLLM_PAGE;
-  const int pps = (pe - pb + 1 + p.n_split - 1) / p.n_split;
-  const int p0 = pb + split * pps, p1 = min(pe + 1, p0 + pps);
-  const int k_lo = max(k_begin, p0 * SLLM_PAGE), k_hi = min(pos + 1, p1 * SLLM_PAGE);
+  const int keep = RAW ? 0 : p.keep;
+  const SeenKeys seen(pos, pos, p.window, keep);
+  const int pps = (seen.pages + p.n_split - 1) / p.n_split;
+  const int p0 = split * pps, p1 = min(seen.pages, p0 + pps);
+  // dense key numbers: this split's range, and the query's own key
+  const int x_pos = pos - seen.skip * SLLM_PAGE;
+  const int k_lo = keep == 0 ? max(k_begin - seen.skip * SLLM_PAGE, p0 * SLLM_PAGE) : p0 * SLLM_PAGE;
+  const int k_hi = min(x_pos + 1, p1 * SLLM_PAGE);
   const int* bt = p.block_table + (size_t)b * p.max_pages;
   const int nrep = p.H / p.G;
   const bf16* rowp = p.q + (size_t)b * p.q_ld;
@@ -766,23 +785,29 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
   const float sc = p.scale * AD_LOG2E;
   const float cap_l2 = p.softcap * AD_LOG2E, cap_in = p.softcap > 0.f ? p.scale / p.softcap : 0.f;
 
+  // whether the query sees the i-th key of the tile at dense number `base`, whose first key is key f of the sequence
+  auto key_ok = [&](int base, int f, int i) -> bool {
+    return base + i >= k_lo && base + i < k_hi && (keep == 0 || f + i >= k_begin || f + i < keep);
+  };
   auto fetch = [&](uint4 (&kr)[2][NJ], uint4 (&vr)[4][NC], int base) {
-    const size_t row0 = ((size_t)bt[base / SLLM_PAGE] * p.G + g) * SLLM_PAGE + (base % SLLM_PAGE);
-    const bf16* kp = p.kpages + row0 * HD;
-    const bf16* vp = p.vpages + row0 * HD;
+    const int f = seen.key(base);                // a tile of 16 keys lies in one page
+    const size_t row0 = ((size_t)bt[f / SLLM_PAGE] * p.G + g) * SLLM_PAGE + (f % SLLM_PAGE);
+    const bf16* kp = p.kpages + row0 * hd;
+    const bf16* vp = p.vpages + row0 * vd;
 #pragma unroll
     for (int u = 0; u < 2; u++) {
-      int key = base + u * 8 + n;
-      bool ok = key >= k_lo && key < k_hi;
+      const bool ok = key_ok(base, f, u * 8 + n);
 #pragma unroll
-      for (int j = 0; j < NJ; j++) kr[u][j] = ok ? ld_dep16_stream(kp + (size_t)(u * 8 + n) * HD + (j * 4 + t) * 8) : zero;
+      for (int j = 0; j < NJ; j++)
+        kr[u][j] = ok && (!TRIM || (j * 4 + t) * 8 < hd) ? ld_dep16_stream(kp + (size_t)(u * 8 + n) * hd + (j * 4 + t) * 8) : zero;
     }
 #pragma unroll
     for (int i = 0; i < 4; i++) {
-      int kk = 2 * t + (i & 1) + (i >> 1) * 8;
-      bool ok = base + kk >= k_lo && base + kk < k_hi;
+      const int kk = 2 * t + (i & 1) + (i >> 1) * 8;
+      const bool ok = key_ok(base, f, kk);
 #pragma unroll
-      for (int c = 0; c < NC; c++) vr[i][c] = ok ? ld_dep16_stream(vp + (size_t)kk * HD + (c * 8 + n) * 8) : zero;
+      for (int c = 0; c < NC; c++)
+        vr[i][c] = ok && (!TRIM || (c * 8 + n) * 8 < vd) ? ld_dep16_stream(vp + (size_t)kk * vd + (c * 8 + n) * 8) : zero;
     }
   };
   // In raw mode (the kernel is part of a model step) the warp's first tile of keys is asked for before the
@@ -791,23 +816,23 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
   // sequences); with grouped queries it changed nothing.
   constexpr int STEP = AD_WARPS * 16;
   const int base0 = (k_lo & ~15) + warp * 16;
-  const bool early = RAW && !p.late && base0 < k_hi && base0 + 16 <= pos;
+  const bool early = RAW && !p.late && base0 < k_hi && base0 + 16 <= x_pos;
   uint4 ka[2][NJ], va[4][NC];
   if (early) fetch(ka, va, base0);
   if (RAW) pdl_wait();
 
   // raw mode: the block whose range holds the query's own position rotates the new key and appends
   // key and value to the cache; after the barrier below they are cached keys like the others
-  if (RAW && p.write_kv && pos >= k_lo && pos < k_hi && threadIdx.x < CH) {
+  if (RAW && p.write_kv && x_pos >= k_lo && x_pos < k_hi && threadIdx.x < CH) {
     int dl = threadIdx.x * 8;
     float kn[8];
-    rope8_raw(rowp + (size_t)(p.H + g) * HD, dl, p.rot, p.interleaved, csr, kn);
-    uint4 vraw = ld_dep16(rowp + (size_t)(p.H + p.G + g) * HD + dl);
+    rope8_raw(rowp + (size_t)(p.H + g) * KD, dl, p.rot, p.interleaved, csr, kn);
+    uint4 vraw = ld_dep16(rowp + (size_t)(p.H + p.G + g) * KD + dl);
     uint4 kraw;
     __nv_bfloat162* kp2 = (__nv_bfloat162*)&kraw;
 #pragma unroll
     for (int j = 0; j < 4; j++) kp2[j] = __floats2bfloat162_rn(kn[2 * j], kn[2 * j + 1]);
-    size_t off = (((size_t)bt[pos / SLLM_PAGE] * p.G + g) * SLLM_PAGE + (pos % SLLM_PAGE)) * HD + dl;
+    size_t off = (((size_t)bt[pos / SLLM_PAGE] * p.G + g) * SLLM_PAGE + (pos % SLLM_PAGE)) * KD + dl;
     *(uint4*)(const_cast<bf16*>(p.kpages) + off) = kraw;
     *(uint4*)(const_cast<bf16*>(p.vpages) + off) = vraw;
   }
@@ -816,8 +841,8 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
     for (int i = threadIdx.x; i < ROWS * CH; i += AD_WARPS * 32) {
       int r = i / CH, dl = (i % CH) * 8;
       uint4 val = zero;
-      if (r0 + r < nrep) {
-        const bf16* head = rowp + (size_t)(g * nrep + r0 + r) * HD;
+      if (r0 + r < nrep && (!TRIM || dl < hd)) {
+        const bf16* head = rowp + (size_t)(g * nrep + r0 + r) * hd;
         if (RAW) {
           float qr[8];
           rope8_raw(head, dl, p.rot, p.interleaved, csr, qr);
@@ -845,6 +870,7 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
     auto attend = [&](uint4 (&kr)[2][NJ], uint4 (&vr)[4][NC], int base) {
+      const int f = seen.key(base);
       float s[2][4];
 #pragma unroll
       for (int u = 0; u < 2; u++) {
@@ -856,9 +882,8 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
         }
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-          int key = base + u * 8 + 2 * t + (e & 1);
           const float sv = p.softcap > 0.f ? cap_l2 * tanhf(s[u][e] * cap_in) : s[u][e] * sc;
-          s[u][e] = (key >= k_lo && key < k_hi) ? sv : -INFINITY;
+          s[u][e] = key_ok(base, f, u * 8 + 2 * t + (e & 1)) ? sv : -INFINITY;
         }
       }
       float mx0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
@@ -910,9 +935,9 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
     // tile's keys and values are in flight while the current tile is multiplied
     int base = base0;
     const bool have = early && r0 == 0;        // the first tile is here already
-    if constexpr (HD >= 128) {
+    if constexpr (KD == 128) {
       // two register buffers used in turn: the next tile is in flight while this one is multiplied.
-      // (At width 64 a tile is too small for that to pay for the registers.)
+      // (At width 64 a tile is too small for that to pay for the registers, at 256 there are none left.)
       uint4 kb[2][NJ], vb[4][NC];
       if (base < k_hi && !have) fetch(ka, va, base);
       while (base < k_hi) {
@@ -953,8 +978,8 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
     }
     __syncthreads();
     const int rows = min(ROWS, nrep - r0);
-    for (int v = threadIdx.x; v < rows * HD; v += AD_WARPS * 32) {
-      int r = v / HD, dd = v % HD;
+    for (int v = threadIdx.x; v < rows * vd; v += AD_WARPS * 32) {
+      int r = v / vd, dd = v % vd;
       float mn = -INFINITY;
 #pragma unroll
       for (int w = 0; w < AD_WARPS; w++) mn = fmaxf(mn, sm_ml[w][r][0]);
@@ -967,16 +992,17 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_mma_kernel(AttnDeco
       }
       if (p.n_split == 1 && p.tickets != nullptr) {        // nothing to merge with: this is the result
         ls = ad_sink_joined(ls, mn, p.sink, g * nrep + r0 + r);
-        p.out[((size_t)b * p.H + g * nrep + r0 + r) * HD + dd] = __float2bfloat16_rn(ls > 0.f ? a / ls : 0.f);
+        const int h = g * nrep + r0 + r;
+        p.out[((size_t)b * p.H + h) * vd + dd] = ad_gated(p, ls > 0.f ? a / ls : 0.f, b, h * vd + dd);
         continue;
       }
-      float* dst = p.part + (((size_t)b * p.H + g * nrep + r0 + r) * p.n_split + split) * (HD + 2);
+      float* dst = p.part + (((size_t)b * p.H + g * nrep + r0 + r) * p.n_split + split) * (vd + 2);
       dst[dd] = a;
-      if (dd == 0) { dst[HD] = mn; dst[HD + 1] = ls; }
+      if (dd == 0) { dst[vd] = mn; dst[vd + 1] = ls; }
     }
     __syncthreads();
   }
-  ad_ticket_merge(p, b, g, nrep, HD);
+  ad_ticket_merge(p, b, g, nrep, vd);
 }
 
 // out[b, h*HD + d] = sum_s acc_s[d] 2^(m_s - M) / sum_s l_s 2^(m_s - M)
@@ -1020,7 +1046,7 @@ static int attn_decode_launch(const AttnDecodeArgs& a, bf16* out, int B, cudaStr
     static const bool scalar_only = getenv("SLLM_DECODE_SCALAR") != nullptr;   // for comparisons
     if (attn_decode_uses_mma(B, a.H, a.G, HD) && !scalar_only) {
       bool up = nrep > 8;
-#define AD_MMA(UPV, RAWV) sllm_launch(attn_decode_mma_kernel<HD, UPV, RAWV>, grid, dim3(AD_WARPS * 32), 0, stream, a)
+#define AD_MMA(UPV, RAWV) sllm_launch(attn_decode_mma_kernel<HD, HD, UPV, RAWV, false>, grid, dim3(AD_WARPS * 32), 0, stream, a)
       if (a.cs != nullptr) e = up ? AD_MMA(true, true) : AD_MMA(false, true);
       else e = up ? AD_MMA(true, false) : AD_MMA(false, false);
 #undef AD_MMA
@@ -1061,7 +1087,7 @@ static int attn_decode_dispatch(const void* q, int q_ld, void* out, const int* s
   if (cos_sin != nullptr && (rot < 2 || rot > hd || (rot % (interleaved ? 8 : 16)) != 0 || tickets == nullptr)) return SLLM_ERR_ARG;
   AttnDecodeArgs a{(const bf16*)q, q_ld, seq_pos0, block_table, max_pages, (const bf16*)kpages, (const bf16*)vpages,
                    (float*)scratch, H, G, window, n_split, scale, (bf16*)out, tickets, (const float2*)cos_sin, rot, interleaved,
-                   write_kv, 0};
+                   write_kv, 0, 0.f, nullptr, hd, hd, 0, nullptr, 0};
   static const int late = getenv("SLLM_DECODE_LATE_KEYS") != nullptr;   // for comparisons
   a.late = late;
   a.softcap = softcap;
@@ -1105,6 +1131,44 @@ SLLM_EXPORT int sllm_attn_decode_capped_bf16(const void* q, int q_ld, void* out,
   if (tickets == nullptr || !attn_decode_uses_mma(B, H, G, hd) || getenv("SLLM_DECODE_SCALAR") != nullptr) return SLLM_ERR_ARG;
   return attn_decode_dispatch(q, q_ld, out, seq_pos0, block_table, max_pages, kpages, vpages, scratch, tickets, B, H, G, hd,
                               window, scale, n_split, stream, nullptr, 0, 0, 0, softcap, sink);
+}
+
+// The general form on the tensor-core kernel: keys hd wide and values vd wide (multiples of 8 up to 256 and 128), any number of
+// query heads per key/value head, a window or chunks, the first `keep` positions kept visible, capped scores, a sink per head,
+// and a gate (bfloat16 logits [B, gate_ld], or null) on the output. Ticket merge as above; `scratch` holds
+// B * H * n_split * (vd + 2) floats.
+SLLM_EXPORT int sllm_attn_decode_general_takes(int hd, int vd) {
+  return hd >= 8 && hd <= 256 && hd % 8 == 0 && vd >= 8 && vd <= 128 && vd % 8 == 0;
+}
+template <int KD, int VD, bool TRIM>
+static int attn_decode_general_launch(const AttnDecodeArgs& a, int B, cudaStream_t stream) {
+  dim3 grid(a.n_split, a.G, B);
+  if (a.H / a.G > 8)
+    return (int)sllm_launch(attn_decode_mma_kernel<KD, VD, true, false, TRIM>, grid, dim3(AD_WARPS * 32), 0, stream, a);
+  return (int)sllm_launch(attn_decode_mma_kernel<KD, VD, false, false, TRIM>, grid, dim3(AD_WARPS * 32), 0, stream, a);
+}
+SLLM_EXPORT int sllm_attn_decode_general_bf16(const void* q, int q_ld, void* out, const int* seq_pos0, const int* block_table,
+                                              int max_pages, const void* kpages, const void* vpages, void* scratch, int* tickets,
+                                              int B, int H, int G, int hd, int vd, int window, int keep, float scale, int n_split,
+                                              float softcap, const float* sink, const void* gate, int gate_ld,
+                                              cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (!sllm_attn_decode_general_takes(hd, vd) || G < 1 || H % G != 0 || n_split < 1 || keep < 0 || (q_ld & 7) || q_ld < H * hd ||
+      (((uintptr_t)q | (uintptr_t)kpages | (uintptr_t)vpages) & 15) || tickets == nullptr || (gate && gate_ld < H * vd))
+    return SLLM_ERR_ARG;
+  AttnDecodeArgs a{(const bf16*)q, q_ld, seq_pos0, block_table, max_pages, (const bf16*)kpages, (const bf16*)vpages,
+                   (float*)scratch, H, G, window, n_split, scale, (bf16*)out, tickets, nullptr, 0, 0, 0, 0, softcap, sink,
+                   hd, vd, keep, (const bf16*)gate, gate_ld};
+  if (hd == 128 && vd == 128) return attn_decode_general_launch<128, 128, false>(a, B, stream);
+  if (hd == 64 && vd == 64) return attn_decode_general_launch<64, 64, false>(a, B, stream);
+  if (vd <= 64) {
+    if (hd <= 64) return attn_decode_general_launch<64, 64, true>(a, B, stream);
+    if (hd <= 128) return attn_decode_general_launch<128, 64, true>(a, B, stream);
+    return attn_decode_general_launch<256, 64, true>(a, B, stream);
+  }
+  if (hd <= 64) return attn_decode_general_launch<64, 128, true>(a, B, stream);
+  if (hd <= 128) return attn_decode_general_launch<128, 128, true>(a, B, stream);
+  return attn_decode_general_launch<256, 128, true>(a, B, stream);
 }
 
 // Rotary positions, cache write and attention of a decode step in one kernel: `qkv` holds the

@@ -1,6 +1,7 @@
 // Kernels around gated mixers and gated side inputs, for float and bfloat16 activations (A):
-//   qk_norm_store    RMS norm of the whole query projection and of the whole key projection (all heads at once),
-//                    rotation by position, queries out, keys and values into the paged cache
+//   qk_norm_store    biases of the projections, RMS norm of queries and keys (per head, or over all heads at once),
+//                    rotation by position, values mixed with an earlier layer's, queries out, keys and values into
+//                    the paged cache
 //   head_gate        attention output of every head times the sigmoid of that head's gate logit
 //   add_cast         residual stream += pending addend; a copy of the stream in the element type
 //   gelu_mul_rows    gelu(a) times a slice of a per-token table row
@@ -20,77 +21,164 @@ __device__ __forceinline__ float gelu_tanh_f(float v) {
   return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
 }
 
-// ------------------------------------------------------------------ query/key norm, rotation, cache write
-// Row t of c (float or A, row stride ld) holds [H query heads of hd | G key heads of hd | G value heads of vd].
-// With qw / kw (norm weights over H * hd and G * hd columns; either may be null) the query part and the key part
-// are each divided by their root mean square over ALL their columns and multiplied by the weight. Then the
-// first `rot` dims of every query and key head turn by the token's position (table cs[pos][i] = (cos, sin);
-// half pairing i with i + rot / 2, or adjacent pairs), queries go to q_out [T, ldq], keys and values to the
-// token's place in the cache pages. G == 0: queries only.
-template <typename A>
-__global__ void __launch_bounds__(256) qk_norm_store_kernel(const void* __restrict__ c, int c_f32, int ld, A* __restrict__ q_out,
-                                                            int ldq, const int* __restrict__ tok_pos,
-                                                            const int* __restrict__ tok_seq, const int* __restrict__ block_table,
-                                                            int max_pages, const float2* __restrict__ cs, A* __restrict__ kpages,
-                                                            A* __restrict__ vpages, int H, int G, int hd, int vd, int rot,
-                                                            int interleaved, const void* __restrict__ qw,
-                                                            const void* __restrict__ kw, int w_f32, float eps) {
-  __shared__ float red[32];
-  int t = blockIdx.x;
-  int pos = tok_pos[t];
-  size_t row = (size_t)t * ld;
-  int QW = H * hd, KW = G * hd;
+// ------------------------------------------------------------------ biases, query/key norm, rotation, value mixing, cache write
+// Row t of c (float or A, row stride ld) holds [H query heads of hd | G key heads of hd | G value heads of vd], to which
+// `bias` (float, the same columns, or null) is added first. With qw / kw (norm weights; either may be null) queries and
+// keys are divided by their root mean square and multiplied by the weight: over ALL the columns of the query part and of
+// the key part (weights of H * hd and G * hd), or with `per_head` over every head by itself (weights of hd, shared by the
+// heads). Then the first `rot` dims of every query and key head turn by the token's position (table cs[pos][i] = (cos, sin);
+// half pairing i with i + rot / 2, or adjacent pairs), queries go to q_out [T, ldq], keys and values to the token's place in
+// the cache pages. Values may be mixed on the way with those an earlier layer projected for the same token, kept in vmix
+// [T, G * vd]: mix_mode 1 writes them there, mode 2 stores (1 - lam) * v + lam * vmix. G == 0: queries only.
+struct QkStoreArgs {
+  const void* c; int c_f32; int ld;
+  const float* bias;
+  void* q_out; int ldq;
+  const int* tok_pos; const int* tok_seq; const int* block_table; int max_pages;
+  const float2* cs;
+  void* kpages; void* vpages;
+  int H, G, hd, vd, rot, interleaved;
+  const void* qw; const void* kw; int w_f32; int per_head; float eps;
+  void* vmix; int mix_mode; float lam;
+};
+
+template <int V> struct Pack { float f[V]; };
+template <int V> __device__ __forceinline__ Pack<V> ld_pack(const float* p) {
+  Pack<V> r;
+  if constexpr (V == 4) { float4 v = *(const float4*)p; r.f[0] = v.x; r.f[1] = v.y; r.f[2] = v.z; r.f[3] = v.w; }
+  else r.f[0] = *p;
+  return r;
+}
+template <int V> __device__ __forceinline__ Pack<V> ld_pack(const bf16* p) {
+  Pack<V> r;
+  if constexpr (V == 4) { float4 v = ld4(p); r.f[0] = v.x; r.f[1] = v.y; r.f[2] = v.z; r.f[3] = v.w; }
+  else r.f[0] = to_f32(*p);
+  return r;
+}
+template <typename A, int V> __device__ __forceinline__ Pack<V> ld_pack_flag(const void* p, int is_f32, size_t i) {
+  return is_f32 ? ld_pack<V>((const float*)p + i) : ld_pack<V>((const A*)p + i);
+}
+template <typename A, int V> __device__ __forceinline__ void st_pack(A* p, const Pack<V>& r) {
+  if constexpr (V == 4) st4(p, make_float4(r.f[0], r.f[1], r.f[2], r.f[3]));
+  else *p = from_f32<A>(r.f[0]);
+}
+
+#define QKS_WARPS 8
+// V elements a lane and access (4 where widths and addresses allow, else 1). A warp takes a head at a time; a head's
+// elements stay in registers between the sum of squares and the stores (heads of up to 512).
+template <typename A, int V>
+__global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreArgs p) {
+  constexpr int NIT = 16 / V;
+  __shared__ float red[2][QKS_WARPS];
+  extern __shared__ float qks_row[];             // with a rotation: hd floats a warp
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int hd = p.hd, vd = p.vd, QW = p.H * hd, KW = p.G * hd;
+  const int pos = p.tok_pos[t];
+  const size_t row = (size_t)t * p.ld;
   float rq = 1.f, rk = 1.f;
-  if (qw) {
-    float ss = 0.f;
-    for (int j = threadIdx.x; j < QW; j += blockDim.x) { float v = ld_flag<A>(c, c_f32, row + j); ss += v * v; }
-    rq = 1.0f / sqrtf(block_sum(ss, red) / (float)QW + eps);
-  }
-  if (kw && G > 0) {
-    float ss = 0.f;
-    for (int j = threadIdx.x; j < KW; j += blockDim.x) { float v = ld_flag<A>(c, c_f32, row + QW + j); ss += v * v; }
-    rk = 1.0f / sqrtf(block_sum(ss, red) / (float)KW + eps);
+  if (!p.per_head && (p.qw || p.kw)) {
+    float sq = 0.f, sk = 0.f;
+    for (int j = threadIdx.x * V; j < QW + KW; j += QKS_WARPS * 32 * V) {
+      Pack<V> x = ld_pack_flag<A, V>(p.c, p.c_f32, row + j);
+      if (p.bias) {
+        Pack<V> b = ld_pack<V>(p.bias + j);
+#pragma unroll
+        for (int i = 0; i < V; i++) x.f[i] += b.f[i];
+      }
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < V; i++) s = fmaf(x.f[i], x.f[i], s);
+      if (j < QW) sq += s; else sk += s;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < QKS_WARPS; w++) { sq += red[0][w]; sk += red[1][w]; }
+    if (p.qw) rq = 1.0f / sqrtf(sq / (float)QW + p.eps);
+    if (p.kw && KW > 0) rk = 1.0f / sqrtf(sk / (float)KW + p.eps);
   }
   size_t page_slot = 0;
-  if (G > 0) {
-    int page = block_table[(size_t)tok_seq[t] * max_pages + pos / SLLM_PAGE];
-    page_slot = (size_t)page * G * SLLM_PAGE + (pos % SLLM_PAGE);       // + g * PAGE, times the head width
+  if (p.G > 0) {
+    int page = p.block_table[(size_t)p.tok_seq[t] * p.max_pages + pos / SLLM_PAGE];
+    page_slot = (size_t)page * p.G * SLLM_PAGE + (pos % SLLM_PAGE);     // + g * PAGE, times the head width
   }
-  int half = rot >> 1;
-  const float2* csr = cs + (size_t)pos * half;
-  // the turning dims, a pair a thread
-  for (int idx = threadIdx.x; idx < (H + G) * half; idx += blockDim.x) {
-    int head = idx / half, i = idx % half;
-    int i0 = interleaved ? 2 * i : i, i1 = interleaved ? 2 * i + 1 : i + half;
-    int col = head * hd;                                               // the key part follows the query part directly
-    bool is_q = head < H;
-    const void* w = is_q ? qw : kw;
-    int wc = is_q ? col : col - QW;
+  const int half = p.rot >> 1;
+  const float2* csr = p.cs + (size_t)pos * half;
+  float* wrow = qks_row + warp * hd;
+  for (int head = warp; head < p.H + p.G; head += QKS_WARPS) {
+    const bool is_q = head < p.H;
+    const int col = head * hd;                                         // the key part follows the query part directly
+    const void* w = is_q ? p.qw : p.kw;
+    const int wc = p.per_head ? 0 : is_q ? col : col - QW;
+    Pack<V> x[NIT];
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < NIT; it++) {
+      const int j = (it * 32 + lane) * V;
+      if (j >= hd) break;
+      x[it] = ld_pack_flag<A, V>(p.c, p.c_f32, row + col + j);
+      if (p.bias) {
+        Pack<V> b = ld_pack<V>(p.bias + col + j);
+#pragma unroll
+        for (int i = 0; i < V; i++) x[it].f[i] += b.f[i];
+      }
+#pragma unroll
+      for (int i = 0; i < V; i++) ss = fmaf(x[it].f[i], x[it].f[i], ss);
+    }
     float r = is_q ? rq : rk;
-    float x0 = ld_flag<A>(c, c_f32, row + col + i0) * r, x1 = ld_flag<A>(c, c_f32, row + col + i1) * r;
-    if (w) { x0 *= load_w(w, w_f32, wc + i0); x1 *= load_w(w, w_f32, wc + i1); }
-    float2 a = csr[i];
-    float r0 = x0 * a.x - x1 * a.y, r1 = x1 * a.x + x0 * a.y;
-    A* dst = is_q ? q_out + (size_t)t * ldq + col : kpages + (page_slot + (size_t)(head - H) * SLLM_PAGE) * hd;
-    dst[i0] = from_f32<A>(r0);
-    dst[i1] = from_f32<A>(r1);
+    if (p.per_head && w) r = 1.0f / sqrtf(warp_sum(ss) / (float)hd + p.eps);
+    A* dst = is_q ? (A*)p.q_out + (size_t)t * p.ldq + col : (A*)p.kpages + (page_slot + (size_t)(head - p.H) * SLLM_PAGE) * hd;
+#pragma unroll
+    for (int it = 0; it < NIT; it++) {
+      const int j = (it * 32 + lane) * V;
+      if (j >= hd) break;
+      if (w) {
+        Pack<V> ww = ld_pack_flag<bf16, V>(w, p.w_f32, wc + j);
+#pragma unroll
+        for (int i = 0; i < V; i++) x[it].f[i] = x[it].f[i] * r * ww.f[i];
+      }
+      if (p.rot > 0) {
+#pragma unroll
+        for (int i = 0; i < V; i++) wrow[j + i] = x[it].f[i];
+      } else {
+        st_pack<A, V>(dst + j, x[it]);
+      }
+    }
+    if (p.rot > 0) {                                                   // a lane turns a pair; the rest passes as it is
+      __syncwarp();
+      for (int i = lane; i < half; i += 32) {
+        const int i0 = p.interleaved ? 2 * i : i, i1 = p.interleaved ? 2 * i + 1 : i + half;
+        const float2 a = csr[i];
+        const float x0 = wrow[i0], x1 = wrow[i1];
+        dst[i0] = from_f32<A>(x0 * a.x - x1 * a.y);
+        dst[i1] = from_f32<A>(x1 * a.x + x0 * a.y);
+      }
+      for (int j = p.rot + lane; j < hd; j += 32) dst[j] = from_f32<A>(wrow[j]);
+      __syncwarp();
+    }
   }
-  // the dims that pass unturned
-  int tail = hd - rot;
-  for (int idx = threadIdx.x; idx < (H + G) * tail; idx += blockDim.x) {
-    int head = idx / tail, j = rot + idx % tail;
-    int col = head * hd;
-    bool is_q = head < H;
-    const void* w = is_q ? qw : kw;
-    float x = ld_flag<A>(c, c_f32, row + col + j) * (is_q ? rq : rk);
-    if (w) x *= load_w(w, w_f32, (is_q ? col : col - QW) + j);
-    A* dst = is_q ? q_out + (size_t)t * ldq + col : kpages + (page_slot + (size_t)(head - H) * SLLM_PAGE) * hd;
-    dst[j] = from_f32<A>(x);
-  }
-  // values as they are
-  for (int idx = threadIdx.x; idx < G * vd; idx += blockDim.x) {
-    int g = idx / vd, j = idx % vd;
-    vpages[(page_slot + (size_t)g * SLLM_PAGE) * vd + j] = from_f32<A>(ld_flag<A>(c, c_f32, row + QW + KW + idx));
+  // values, one pass of the block over all heads
+  A* vm = (A*)p.vmix + (size_t)t * p.G * vd;
+  for (int e = threadIdx.x * V; e < p.G * vd; e += QKS_WARPS * 32 * V) {
+    const int g = e / vd, j = e % vd;
+    Pack<V> x = ld_pack_flag<A, V>(p.c, p.c_f32, row + QW + KW + e);
+    if (p.bias) {
+      Pack<V> b = ld_pack<V>(p.bias + QW + KW + e);
+#pragma unroll
+      for (int i = 0; i < V; i++) x.f[i] += b.f[i];
+    }
+    if (p.mix_mode == 1) st_pack<A, V>(vm + e, x);
+    if (p.mix_mode == 2) {
+      Pack<V> f = ld_pack<V>((const A*)vm + e);
+#pragma unroll
+      for (int i = 0; i < V; i++) x.f[i] = (1.0f - p.lam) * x.f[i] + p.lam * f.f[i];
+    }
+    st_pack<A, V>((A*)p.vpages + (page_slot + (size_t)g * SLLM_PAGE) * vd + j, x);
   }
 }
 
@@ -430,24 +518,28 @@ __global__ void gelu_mul_rows_kernel(const A* __restrict__ a, int lda, const int
   out[i] = from_f32<A>(gelu_tanh_f(to_f32(a[(size_t)t * lda + j])) * e);
 }
 
-// ------------------------------------------------------------------ x += y / rms(y) * w
-// y float or A: [P][T][d] partial sums added in their order; a block per row, the row's y kept in shared memory.
+// ------------------------------------------------------------------ x += (y + yb) / rms(y + yb) * w
+// y float or A: [P][T][d] partial sums added in their order, then yb (float [d], the product's bias, or null); a block per
+// row, the row's y kept in shared memory.
 // With `out` (A, [gridDim.x][d]) the row's norm for the next reader follows in the same pass: out = x / rms(x) * w2 of
 // the stream as it now stands, or with `b2` the norm without statistics tanh(alpha2 x) * w2 + b2 (w2, b2 float then);
-// `rows` (or null) picks the stream's rows that are worked on, out's rows stay in order. `vec` (float [d], or null)
-// is added to the row as well.
+// without w2 it is the stream's row itself in the element type. `rows` (or null) picks the stream's rows that are worked on,
+// out's rows stay in order. `vec` (float [d], or null) is added to the row as well.
 template <typename A>
-__global__ void add_rms_normed_kernel(float* __restrict__ x, const void* __restrict__ y, int y_f32, int P, int T,
+__global__ void add_rms_normed_kernel(float* x, const void* y, int y_f32, int P, int T, const float* yb,
                                       const void* __restrict__ w, int w_f32, int d, float eps, const int* __restrict__ rows,
-                                      const void* __restrict__ w2, int w2_f32, float eps2, A* __restrict__ out,
+                                      const void* __restrict__ w2, int w2_f32, float eps2, A* out,
                                       const float* __restrict__ vec, const float* __restrict__ b2, float alpha2) {
   extern __shared__ __align__(16) float rowbuf[];
   __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
   int t = rows ? rows[blockIdx.x] : blockIdx.x;
   float ss = 0.f;
   for (int j = threadIdx.x; j < d; j += blockDim.x) {
     float v = 0.f;
     for (int p = 0; p < P; p++) v += ld_flag<A>(y, y_f32, ((size_t)p * T + t) * d + j);
+    if (yb) v += yb[j];
     rowbuf[j] = v;
     ss += v * v;
   }
@@ -457,10 +549,11 @@ __global__ void add_rms_normed_kernel(float* __restrict__ x, const void* __restr
     float v = x[(size_t)t * d + j] + rowbuf[j] * r * load_w(w, w_f32, j);
     if (vec) v += vec[j];
     x[(size_t)t * d + j] = v;
+    if (out && !w2) out[(size_t)blockIdx.x * d + j] = from_f32<A>(v);
     rowbuf[j] = v;                             // a column is one thread's in every pass
     ss2 += v * v;
   }
-  if (!out) return;
+  if (!out || !w2) return;
   if (b2) {
     for (int j = threadIdx.x; j < d; j += blockDim.x)
       out[(size_t)blockIdx.x * d + j] = from_f32<A>(tanhf(alpha2 * rowbuf[j]) * load_w(w2, 1, j) + b2[j]);
@@ -473,12 +566,14 @@ __global__ void add_rms_normed_kernel(float* __restrict__ x, const void* __restr
 
 // four columns a thread (d a multiple of four); the partial sums are added in the same order
 template <typename A>
-__global__ void add_rms_normed_vec_kernel(float* __restrict__ x, const void* __restrict__ y, int y_f32, int P, int T,
+__global__ void add_rms_normed_vec_kernel(float* x, const void* y, int y_f32, int P, int T, const float* yb,
                                           const void* __restrict__ w, int w_f32, int d, float eps, const int* __restrict__ rows,
-                                          const void* __restrict__ w2, int w2_f32, float eps2, A* __restrict__ out,
+                                          const void* __restrict__ w2, int w2_f32, float eps2, A* out,
                                           const float* __restrict__ vec, const float* __restrict__ b2, float alpha2) {
   extern __shared__ __align__(16) float rowbuf[];
   __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
   int t = rows ? rows[blockIdx.x] : blockIdx.x;
   float ss = 0.f;
   for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
@@ -486,6 +581,10 @@ __global__ void add_rms_normed_vec_kernel(float* __restrict__ x, const void* __r
     for (int p = 0; p < P; p++) {
       float4 a = ld4f<A>(y, y_f32, ((size_t)p * T + t) * d + j);
       v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+    }
+    if (yb) {
+      float4 b = *(const float4*)(yb + j);
+      v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
     }
     *(float4*)(rowbuf + j) = v;
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -504,10 +603,11 @@ __global__ void add_rms_normed_vec_kernel(float* __restrict__ x, const void* __r
       xv.x += b.x; xv.y += b.y; xv.z += b.z; xv.w += b.w;
     }
     *(float4*)(x + (size_t)t * d + j) = xv;
+    if (out && !w2) { st4(out + (size_t)blockIdx.x * d + j, xv); continue; }
     *(float4*)(rowbuf + j) = xv;
     ss2 += xv.x * xv.x + xv.y * xv.y + xv.z * xv.z + xv.w * xv.w;
   }
-  if (!out) return;
+  if (!out || !w2) return;
   if (b2) {
     for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
       float4 v = *(const float4*)(rowbuf + j);

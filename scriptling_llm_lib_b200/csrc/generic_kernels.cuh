@@ -28,6 +28,32 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const W* __restri
   for (int j = threadIdx.x; j < d; j += blockDim.x) dst[j] = ok ? to_f32(src[j]) : 0.f;
 }
 
+// The embedding with a vector per position: out[t, 2i] = table[ids[t], 2i] + sin(pos f_i), out[t, 2i + 1] = ... + cos(pos f_i).
+// The host hands over (sin, cos) of 64 a f_i (`coarse`, [positions / 64][pairs]) and of b f_i (`fine`, [64][pairs]), made in
+// double and rounded once, and pos = 64 a + b is put together here by the addition theorem: float sums of products of
+// numbers of at most 1, an error of about 1e-7 at any position. A position past the tables raises *err.
+template <typename W>
+__global__ void embed_rows_sinusoid_kernel(const int* __restrict__ ids, const int* __restrict__ tok_pos, const W* __restrict__ table,
+                                           const float2* __restrict__ coarse, const float2* __restrict__ fine,
+                                           float* __restrict__ out, int d, int vocab, int n_coarse, int* err) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, id = ids[t], pos = tok_pos[t], pairs = (d + 1) >> 1;
+  const bool ok = id >= 0 && id < vocab && (pos >> 6) < n_coarse;
+  if (!ok && threadIdx.x == 0) atomicExch(err, 1);
+  const W* src = table + (size_t)(ok ? id : 0) * d;
+  const float2* ca = coarse + (size_t)(ok ? pos >> 6 : 0) * pairs;
+  const float2* fb = fine + (size_t)(pos & 63) * pairs;
+  float* dst = out + (size_t)t * d;
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const float2 a = ca[i], b = fb[i];
+    const float s = a.x * b.y + a.y * b.x, c = a.y * b.y - a.x * b.x;
+    const int j = 2 * i;
+    dst[j] = ok ? to_f32(src[j]) + s : 0.f;
+    if (j + 1 < d) dst[j + 1] = ok ? to_f32(src[j + 1]) + c : 0.f;
+  }
+}
+
 // The embedding with a second table looked up by the pair (previous token, token):
 // out[t, :] = table[ids[t], :] + pair_table[r, :], r = (prev * mul_prev + ids[t] * mul_cur) mod buckets, and r = buckets (the
 // table's last row) for a sequence's first token (tok_pos 0). The previous token of a step's row is the row before it; for
@@ -531,7 +557,8 @@ __global__ void rope_kv_write_vec_kernel(A* __restrict__ qkv, int ld, const int*
 // ------------------------------------------------------------------ attention over the paged cache
 // One block: ATT_BQ consecutive queries of one sequence, one query head. Keys and values come
 // from the cache (this step's own keys were written before). Key j is seen by the query at
-// absolute position p when j <= p and (window == 0 or j > p - window). Online softmax in float:
+// absolute position p when j <= p and (window == 0 or j > p - window), or j < keep (the sequence's first positions,
+// which stay visible behind any window). Values may have a width of their own (vd). Online softmax in float:
 // running maximum m, running sum l, accumulator rescaled when m grows.
 #define ATT_BQ 16
 #define ATT_BK 32
@@ -547,14 +574,14 @@ __device__ __forceinline__ float sink_joined(float l, float m, float sink) {
 struct AttnArgs {
   const void* q;        // [T, q_ld] rotated queries; head h at columns h*hd
   int q_ld;
-  void* out;            // [T, H*hd]
+  void* out;            // [T, H*vd]
   const int* seq_start; // [B+1] first row of each sequence in the packed batch
   const int* seq_pos0;  // [B] cache length of each sequence before this step
   const int* block_table;
   int max_pages;
   const void* kpages;   // [pages][G][PAGE][hd]
-  const void* vpages;
-  int H, G, hd, window;
+  const void* vpages;   // [pages][G][PAGE][vd]
+  int H, G, hd, vd, window, keep;
   float scale;
   float softcap;        // > 0: a score s becomes softcap * tanh(s / softcap) before the softmax
   const float* sink;    // [H] or null: exp(sink[h]) joins the softmax's denominator, with no key and no value
@@ -563,10 +590,10 @@ struct AttnArgs {
 template <typename A, int NACC>
 __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
   extern __shared__ float att_sm[];
-  const int hd = p.hd;
+  const int hd = p.hd, vd = p.vd;
   float* Qs = att_sm;                          // [ATT_BQ][hd]
   float* Ks = Qs + ATT_BQ * hd;                // [ATT_BK][hd + 1]
-  float* Vs = Ks + ATT_BK * (hd + 1);          // [ATT_BK][hd]
+  float* Vs = Ks + ATT_BK * (hd + 1);          // [ATT_BK][vd]
   int b = blockIdx.z, h = blockIdx.y, qt = blockIdx.x;
   int row0 = p.seq_start[b], S = p.seq_start[b + 1] - row0;
   int r0 = qt * ATT_BQ;
@@ -595,20 +622,21 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
   }
 
   int k_hi = pos0 + r0 + nq;                                   // one past the last key any query sees
-  int k_lo = first_seen(pos0 + r0, p.window);
-  k_lo = (k_lo / ATT_BK) * ATT_BK;
+  const SeenKeys seen_keys(pos0 + r0, k_hi - 1, p.window, p.keep);
   const int* bt = p.block_table + (size_t)b * p.max_pages;
 
-  for (int kt = k_lo; kt < k_hi; kt += ATT_BK) {
+  for (int x = 0; x < seen_keys.pages * SLLM_PAGE; x += ATT_BK) {
+    const int kt = seen_keys.key(x);
+    if (kt >= k_hi) break;
     int page = bt[kt / SLLM_PAGE];
-    size_t base = ((size_t)page * p.G + g) * SLLM_PAGE * hd + (size_t)(kt % SLLM_PAGE) * hd;
+    size_t row = ((size_t)max(page, 0) * p.G + g) * SLLM_PAGE + (size_t)(kt % SLLM_PAGE);
     __syncthreads();
     for (int e = threadIdx.x; e < ATT_BK * hd; e += ATT_THREADS) {
       int kk = e / hd, dd = e % hd;
-      bool ok = page >= 0 && (kt + kk) < k_hi;
-      Ks[kk * (hd + 1) + dd] = ok ? to_f32(kp[base + e]) : 0.f;
-      Vs[e] = ok ? to_f32(vp[base + e]) : 0.f;
+      Ks[kk * (hd + 1) + dd] = page >= 0 && (kt + kk) < k_hi ? to_f32(kp[row * hd + e]) : 0.f;
     }
+    for (int e = threadIdx.x; e < ATT_BK * vd; e += ATT_THREADS)
+      Vs[e] = page >= 0 && (kt + e / vd) < k_hi ? to_f32(vp[row * vd + e]) : 0.f;
     __syncthreads();
     int kpos = kt + lane;
 #pragma unroll
@@ -622,7 +650,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
       for (int dd = 0; dd < hd; dd++) dot = fmaf(qv[dd], kv[dd], dot);
       float s = dot * p.scale;
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
-      bool seen = page >= 0 && kpos <= qpos && kpos >= first_seen(qpos, p.window);
+      bool seen = page >= 0 && key_seen(kpos, qpos, first_seen(qpos, p.window), p.keep);
       if (!seen) s = -INFINITY;
       float m_new = fmaxf(m[i], warp_max(s));
       if (m_new == -INFINITY) continue;                        // nothing seen yet by this query
@@ -637,7 +665,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
 #pragma unroll
         for (int a = 0; a < NACC; a++) {
           int dd = lane + 32 * a;
-          if (dd < hd) acc[i][a] = fmaf(pk, Vs[kk * hd + dd], acc[i][a]);
+          if (dd < vd) acc[i][a] = fmaf(pk, Vs[kk * vd + dd], acc[i][a]);
         }
       }
     }
@@ -652,7 +680,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
 #pragma unroll
     for (int a = 0; a < NACC; a++) {
       int dd = lane + 32 * a;
-      if (dd < hd) out[(size_t)(row0 + r0 + qi) * ((size_t)p.H * hd) + (size_t)h * hd + dd] = from_f32<A>(acc[i][a] * inv);
+      if (dd < vd) out[(size_t)(row0 + r0 + qi) * ((size_t)p.H * vd) + (size_t)h * vd + dd] = from_f32<A>(acc[i][a] * inv);
     }
   }
 }
@@ -665,7 +693,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
 // kept k-major (transposed: Qs[d][query], Ks[d][key]), the values row-major, the probabilities
 // row-major with a padded stride. Softmax statistics live in registers, the row maximum and sum are
 // folded over the 16 lanes that share a query. The same mathematics and masks as the kernel above;
-// head widths in multiples of 4 up to 64 * NG.
+// key and value widths in multiples of 4, values up to 64 * NG.
 #define ATT2_BQ 64
 #define ATT2_BK 64
 #define ATT2_PS (ATT2_BK + 4)
@@ -673,11 +701,11 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_paged_kernel(AttnArgs p) {
 template <typename A, int NG>
 __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
   extern __shared__ __align__(16) float att_sm[];
-  const int hd = p.hd;
+  const int hd = p.hd, vd = p.vd;
   float* Qs = att_sm;                          // [hd][64]
   float* Ks = Qs + hd * ATT2_BQ;               // [hd][64]
-  float* Vs = Ks + hd * ATT2_BK;               // [64][hd]
-  float* Ps = Vs + ATT2_BK * hd;               // [64][68]
+  float* Vs = Ks + hd * ATT2_BK;               // [64][vd]
+  float* Ps = Vs + ATT2_BK * vd;               // [64][68]
   const int b = blockIdx.z, h = blockIdx.y, qt = blockIdx.x;
   const int row0 = p.seq_start[b], S = p.seq_start[b + 1] - row0;
   const int r0 = qt * ATT2_BQ;
@@ -689,7 +717,7 @@ __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
   const A* q = (const A*)p.q;
   const A* kp = (const A*)p.kpages;
   const A* vp = (const A*)p.vpages;
-  const int vec_per_row = hd >> 2;
+  const int vec_per_row = hd >> 2, vvec_per_row = vd >> 2;
 
   for (int e = tid; e < ATT2_BQ * vec_per_row; e += 256) {
     int qi = e % ATT2_BQ, dq = e / ATT2_BQ;
@@ -709,26 +737,26 @@ __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
       for (int c = 0; c < 4; c++) o[i][gg][c] = 0.f;
   }
   const int k_hi = pos0 + r0 + nq;
-  int k_lo = first_seen(pos0 + r0, p.window);
-  k_lo = (k_lo / ATT2_BK) * ATT2_BK;
+  const SeenKeys seen_keys(pos0 + r0, k_hi - 1, p.window, p.keep);
   const int* bt = p.block_table + (size_t)b * p.max_pages;
 
-  for (int kt = k_lo; kt < k_hi; kt += ATT2_BK) {
+  for (int v = 0; v < seen_keys.pages; v++) {
+    const int kt = seen_keys.page(v) * ATT2_BK;
     const int page = bt[kt / SLLM_PAGE];               // a tile is one page (both are 64 keys)
-    const size_t base = ((size_t)max(page, 0) * p.G + g) * SLLM_PAGE * hd;
+    const size_t row = ((size_t)max(page, 0) * p.G + g) * SLLM_PAGE;
     __syncthreads();
     for (int e = tid; e < ATT2_BK * vec_per_row; e += 256) {
       int kk = e % ATT2_BK, dq = e / ATT2_BK;
       bool ok = page >= 0 && kt + kk < k_hi;
-      float4 v = ok ? ld4(kp + base + (size_t)kk * hd + dq * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      float4 v = ok ? ld4(kp + (row + kk) * hd + dq * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
       Ks[(dq * 4 + 0) * ATT2_BK + kk] = v.x; Ks[(dq * 4 + 1) * ATT2_BK + kk] = v.y;
       Ks[(dq * 4 + 2) * ATT2_BK + kk] = v.z; Ks[(dq * 4 + 3) * ATT2_BK + kk] = v.w;
     }
-    for (int e = tid; e < ATT2_BK * vec_per_row; e += 256) {
-      int kk = e / vec_per_row, dq = e % vec_per_row;
+    for (int e = tid; e < ATT2_BK * vvec_per_row; e += 256) {
+      int kk = e / vvec_per_row, dq = e % vvec_per_row;
       bool ok = page >= 0 && kt + kk < k_hi;
-      float4 v = ok ? ld4(vp + base + (size_t)kk * hd + dq * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-      *(float4*)(Vs + kk * hd + dq * 4) = v;
+      float4 v = ok ? ld4(vp + (row + kk) * vd + dq * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      *(float4*)(Vs + kk * vd + dq * 4) = v;
     }
     __syncthreads();
     float s[4][4];
@@ -753,7 +781,7 @@ __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
 #pragma unroll
       for (int j = 0; j < 4; j++) {
         int kpos = kt + tx * 4 + j;
-        bool seen = page >= 0 && qi < nq && kpos <= qpos && kpos >= first_seen(qpos, p.window);
+        bool seen = page >= 0 && qi < nq && key_seen(kpos, qpos, first_seen(qpos, p.window), p.keep);
         s[i][j] = seen ? capped(s[i][j] * p.scale, p.softcap) : -INFINITY;
         mx = fmaxf(mx, s[i][j]);
       }
@@ -787,10 +815,10 @@ __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
 #pragma unroll
       for (int gg = 0; gg < NG; gg++) {
         const int d0 = (tx + 16 * gg) * 4;
-        if (d0 >= hd) continue;
+        if (d0 >= vd) continue;
 #pragma unroll
         for (int kk = 0; kk < 4; kk++) {
-          float4 vv = *(const float4*)(Vs + (k4 + kk) * hd + d0);
+          float4 vv = *(const float4*)(Vs + (k4 + kk) * vd + d0);
 #pragma unroll
           for (int i = 0; i < 4; i++) {
             o[i][gg][0] = fmaf(pv[i][kk], vv.x, o[i][gg][0]);
@@ -815,8 +843,8 @@ __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
 #pragma unroll
     for (int gg = 0; gg < NG; gg++) {
       const int d0 = (tx + 16 * gg) * 4;
-      if (d0 >= hd) continue;
-      st4(out + (size_t)(row0 + r0 + qi) * ((size_t)p.H * hd) + (size_t)h * hd + d0,
+      if (d0 >= vd) continue;
+      st4(out + (size_t)(row0 + r0 + qi) * ((size_t)p.H * vd) + (size_t)h * vd + d0,
           make_float4(o[i][gg][0] * inv, o[i][gg][1] * inv, o[i][gg][2] * inv, o[i][gg][3] * inv));
     }
   }
@@ -828,18 +856,19 @@ __global__ void __launch_bounds__(256) attn_paged_tiled_kernel(AttnArgs p) {
 // heads: once per NREP of them), LPK lanes per key with 4 dims each per pass (NV passes for wide
 // heads), online softmax per lane group and head in float (exponentials as 2^x of scores scaled by
 // log2 e), folded over the warp and the block. With one split the block writes the output row; otherwise it leaves
-// (unnormalised sum, maximum, sum) in `part` [B][H][n_split][hd + 2] for the merge kernel below.
+// (unnormalised sum, maximum, sum) in `part` [B][H][n_split][vd + 2] for the merge kernel below.
+// Keys and values may have different widths, both up to LPK * 4 * NV.
 struct AttnSplitArgs {
   const void* q;        // [B, q_ld] rotated queries of this step
   int q_ld;
-  void* out;            // [B, H*hd]
+  void* out;            // [B, H*vd]
   const int* seq_pos0;  // [B] position of the query: the cache holds keys 0..pos
   const int* block_table;
   int max_pages;
   const void* kpages;
   const void* vpages;
   float* part;
-  int H, G, hd, window, n_split;
+  int H, G, hd, vd, window, keep, n_split;
   float scale;
   float softcap;        // as in AttnArgs
   const float* sink;
@@ -850,23 +879,23 @@ template <typename A, int LPK, int NV, int NREP>
 __global__ void __launch_bounds__(128) attn_decode_split_generic_kernel(AttnSplitArgs p) {
   constexpr int KPW = 32 / LPK;                 // keys a warp reads per load
   constexpr int UN = NV == 1 ? 4 : (NV == 2 ? 2 : 1);   // loads in flight per lane group
-  extern __shared__ __align__(16) float ad_sm[];        // [4 warps][NREP][hd] partial outputs, then [4][NREP][2] (m, l)
-  const int hd = p.hd;
+  extern __shared__ __align__(16) float ad_sm[];        // [4 warps][NREP][vd] partial outputs, then [4][NREP][2] (m, l)
+  const int hd = p.hd, vd = p.vd;
   const int split = blockIdx.x, g = blockIdx.y, b = blockIdx.z;
   const int nrep = p.H / p.G;                   // query heads that share this key/value head: served NREP at a time
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int slot = lane / LPK, dl = (lane % LPK) * 4;
   const int pos = p.seq_pos0[b];
   const int k_begin = first_seen(pos, p.window);
-  const int pb = k_begin / SLLM_PAGE, pe = pos / SLLM_PAGE;
-  const int pps = (pe - pb + p.n_split) / p.n_split;
-  const int p0 = pb + split * pps, p1 = min(pe + 1, p0 + pps);
-  const int k_lo = max(k_begin, p0 * SLLM_PAGE), k_hi = min(pos + 1, p1 * SLLM_PAGE);
+  const SeenKeys seen_keys(pos, pos, p.window, p.keep);
+  const int pps = (seen_keys.pages + p.n_split - 1) / p.n_split;
+  const int p0 = split * pps, p1 = min(seen_keys.pages, p0 + pps);
+  const int x_lo = p0 * SLLM_PAGE, x_hi = p1 * SLLM_PAGE;      // dense key numbers of this split
   const int* bt = p.block_table + (size_t)b * p.max_pages;
   const A* kp = (const A*)p.kpages;
   const A* vp = (const A*)p.vpages;
-  float* sm_acc = ad_sm;                        // [4][NREP][hd]
-  float* sm_ml = ad_sm + 4 * NREP * hd;         // [4][NREP][2]
+  float* sm_acc = ad_sm;                        // [4][NREP][vd]
+  float* sm_ml = ad_sm + 4 * NREP * vd;         // [4][NREP][2]
 
   for (int r0 = 0; r0 < nrep; r0 += NREP) {
     float qv[NREP][NV][4], acc[NREP][NV][4], m[NREP], l[NREP];
@@ -885,21 +914,25 @@ __global__ void __launch_bounds__(128) attn_decode_split_generic_kernel(AttnSpli
       m[r] = -INFINITY;
       l[r] = 0.f;
     }
-    for (int kb = k_lo + warp * KPW * UN; kb < k_hi; kb += 4 * KPW * UN) {
+    for (int kb = x_lo + warp * KPW * UN; kb < x_hi; kb += 4 * KPW * UN) {
+      {                                         // keys no query sees: the ends of the kept and of the window's first page
+        const int f = seen_keys.key(kb);
+        if (f > pos || (f >= p.keep && f + KPW * UN <= k_begin)) continue;
+      }
       float4 kr[UN][NV], vr[UN][NV];
       bool ok[UN];
 #pragma unroll
       for (int u = 0; u < UN; u++) {
-        int key = kb + u * KPW + slot;
-        ok[u] = key < k_hi;
-        int kk = ok[u] ? key : k_lo;
+        int key = seen_keys.key(kb + u * KPW + slot);
+        ok[u] = key_seen(key, pos, k_begin, p.keep);
+        int kk = ok[u] ? key : pos;
         int page = bt[kk / SLLM_PAGE];
-        size_t off = (((size_t)page * p.G + g) * SLLM_PAGE + (kk % SLLM_PAGE)) * hd;
+        size_t row = ((size_t)page * p.G + g) * SLLM_PAGE + (kk % SLLM_PAGE);
 #pragma unroll
         for (int v = 0; v < NV; v++) {
           int d = dl + v * LPK * 4;
-          kr[u][v] = d < hd ? ld4(kp + off + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-          vr[u][v] = d < hd ? ld4(vp + off + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+          kr[u][v] = d < hd ? ld4(kp + row * hd + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+          vr[u][v] = d < vd ? ld4(vp + row * vd + d) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
       }
 #pragma unroll
@@ -959,14 +992,14 @@ __global__ void __launch_bounds__(128) attn_decode_split_generic_kernel(AttnSpli
 #pragma unroll
         for (int v = 0; v < NV; v++) {
           int d = dl + v * LPK * 4;
-          if (d < hd) *(float4*)(sm_acc + (warp * NREP + r) * hd + d) = make_float4(acc[r][v][0], acc[r][v][1], acc[r][v][2], acc[r][v][3]);
+          if (d < vd) *(float4*)(sm_acc + (warp * NREP + r) * vd + d) = make_float4(acc[r][v][0], acc[r][v][1], acc[r][v][2], acc[r][v][3]);
         }
         if (lane == 0) { sm_ml[(warp * NREP + r) * 2] = m[r]; sm_ml[(warp * NREP + r) * 2 + 1] = l[r]; }
       }
     }
     __syncthreads();
-    for (int e = threadIdx.x; e < NREP * hd; e += 128) {
-      const int r = e / hd, dd = e % hd;
+    for (int e = threadIdx.x; e < NREP * vd; e += 128) {
+      const int r = e / vd, dd = e % vd;
       if (r0 + r >= nrep) continue;
       const int h = g * nrep + r0 + r;
       float mn = -INFINITY;
@@ -976,16 +1009,16 @@ __global__ void __launch_bounds__(128) attn_decode_split_generic_kernel(AttnSpli
 #pragma unroll
       for (int w = 0; w < 4; w++) {
         float cw = mn == -INFINITY ? 0.f : exp2f(sm_ml[(w * NREP + r) * 2] - mn);
-        a += sm_acc[(w * NREP + r) * hd + dd] * cw;
+        a += sm_acc[(w * NREP + r) * vd + dd] * cw;
         ls += sm_ml[(w * NREP + r) * 2 + 1] * cw;
       }
       if (p.n_split == 1) {
         if (p.sink) ls = mn == -INFINITY ? 1.0f : ls + exp2f(p.sink[h] * ATT_LOG2E - mn);
-        ((A*)p.out)[((size_t)b * p.H + h) * hd + dd] = from_f32<A>(ls > 0.f ? a / ls : 0.f);
+        ((A*)p.out)[((size_t)b * p.H + h) * vd + dd] = from_f32<A>(ls > 0.f ? a / ls : 0.f);
       } else {
-        float* dst = p.part + (((size_t)b * p.H + h) * p.n_split + split) * (hd + 2);
+        float* dst = p.part + (((size_t)b * p.H + h) * p.n_split + split) * (vd + 2);
         dst[dd] = a;
-        if (dd == 0) { dst[hd] = mn; dst[hd + 1] = ls; }
+        if (dd == 0) { dst[vd] = mn; dst[vd + 1] = ls; }
       }
     }
     __syncthreads();

@@ -102,6 +102,12 @@ class StepContext:
         return self.kernels.decode.attention_splits(self.n_seqs, n_heads, n_kv_heads, head_dim, self.max_pages,
                                                     self.engine.sm_count)
 
+    def pages_seen(self, unit: int) -> int:
+        """The most pages a query of this step sees in the unit: its sequence's, or what the unit's window and kept first
+        positions come to."""
+        bound = self.cache.groups[self.cache.group_of_unit[unit]].need.pages_seen()
+        return self.max_pages if bound is None else max(1, min(self.max_pages, bound))
+
     def unit_kv(self, unit: int):
         g = self.cache.group_of_unit[unit]
         k, v = self.cache.groups[g].unit_storage(unit)

@@ -36,6 +36,18 @@ concatenated heads are multiplied element by element with the sigmoid of its pro
 (both precisions; scores, cap, softmax and sink float32) and, in bfloat16 with heads of 64 or 128, to the tcgen05 prompt
 kernels and to the decode kernel that puts a group's query heads on the tensor cores.
 
+Five more, none in the reference. `keep_first`: the first positions of a sequence stay visible behind the window, at their
+true positions; the cache keeps their pages. `biases`: stored vectors added to the projected queries, keys and values
+(in the store kernel) and to the output product (`o_name`; the mixer then answers with the output and the vector, a
+`WithRowVector`, and the next reader of the stream adds both). `qk_norm` with `per="head"`: every query and key head is
+divided by its own root mean square and multiplied by a weight of one head's width, shared by the heads. `sink_value`: the
+same sink logit for every head as a constant instead of a stored one (0: one is added to the denominator). `value_mix`:
+layers that share a `group` mix their values with those the group's first layer projected for the same token, v <- (1 - lam)
+v + lam v_first with lam a stored number, before they are cached; the first layer's values stay at hand for the step.
+With any of these, attention runs on the kernels that know keys and values of different widths, the window with kept
+positions and the sink: in bfloat16 the tcgen05 prompt kernels (heads of 64 and 128), the mma.sync prompt and decode
+kernels (keys up to 256, values up to 128, multiples of 8), else and in 32-bit the generic ones.
+
 The position encoding is optional (`position=None`: queries and keys as projected). Storing keys
 and values in the cache is this mixer's own step, whatever the encoding: for an encoding that is a
 rotation by a table the store and the rotation are one kernel (or part of the q|k|v product's
@@ -49,12 +61,13 @@ import math
 import torch
 
 from ..cache.needs import CacheNeed
-from ..csrc.bindings import DecodeKernels, PrefillAttentionTC
+from ..csrc.bindings import DecodeKernels, PrefillAttentionMMA, PrefillAttentionTC, gate_aligned
 from ..cache.needs import StateNeed
 from ..weights.spec import TensorSpec
 from .base import MIXERS, POSITION_ENCODINGS, Folded, Mixer, PartSpec
 from .conv import CausalConv
 from .linear import Linear
+from .norm import WithRowVector
 
 
 class Attention(Mixer):
@@ -69,7 +82,8 @@ class Attention(Mixer):
                  scale: float | None = None, v_dim: int | None = None, value_norm_eps: float | None = None,
                  chunk: int | None = None, conv: dict | None = None, qk_norm: dict | None = None, gate_name: str | None = None,
                  values_are_keys: bool = False, softcap: float | None = None, sink_name: str | None = None,
-                 gate_per: str = "head"):
+                 gate_per: str = "head", keep_first: int = 0, biases: dict | None = None, sink_value: float | None = None,
+                 value_mix: dict | None = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads cannot share {n_kv_heads} key/value heads")
         if not 1 <= head_dim <= 512:
@@ -91,9 +105,25 @@ class Attention(Mixer):
         if self.softcap is not None and not self.softcap > 0:
             raise ValueError(f"a cap on the scores must be positive, got {softcap}")
         self.sink_name, self.sink = sink_name, None
-        self.plain_softmax = self.softcap is None and sink_name is None
-        if not self.plain_softmax and v_dim is not None and int(v_dim) != head_dim:
-            raise ValueError("capped scores and sinks run on kernels whose values are as wide as the keys")
+        if sink_name is not None and sink_value is not None:
+            raise ValueError("a head's sink is stored or a constant, not both")
+        self.sink_value = None if sink_value is None else float(sink_value)
+        self.plain_softmax = self.softcap is None and sink_name is None and sink_value is None
+        self.keep_first = int(keep_first)
+        if self.keep_first < 0 or (self.keep_first and not window):
+            raise ValueError("the first positions are kept visible behind a sliding window")
+        self.bias_names = dict(biases) if biases else {}
+        if self.bias_names and (conv is not None or self.values_are_keys):
+            raise ValueError("projections with biases take neither a convolution nor values that are the keys")
+        if self.bias_names and not {"q_name", "k_name", "v_name"} <= set(self.bias_names):
+            raise ValueError("queries, keys and values have biases, or none of them has")
+        self.in_bias = self.out_bias = None
+        self.value_mix = dict(value_mix) if value_mix else None
+        self.mix_share = None
+        if value_norm_eps is not None and (conv is not None or qk_norm is not None or gate_name is not None or biases or value_mix
+                                           or keep_first or not self.plain_softmax):
+            raise ValueError("a value norm goes with none of convolution, query/key norm, gate, biases, mixed values, kept "
+                             "positions, cap and sink")
         self.gate_per = gate_per
         self.hidden, self.n_heads, self.n_kv_heads, self.head_dim, self.window = hidden, n_heads, n_kv_heads, head_dim, window
         self.chunk = int(chunk) if chunk else None
@@ -118,12 +148,19 @@ class Attention(Mixer):
         if conv is not None and int(conv["taps"]) > 1:
             self.conv = CausalConv([conv["q_name"], conv["k_name"], conv["v_name"]], [qw, kw, vw], int(conv["taps"]))
         self.qk_norm = dict(qk_norm) if qk_norm is not None else None
+        self.norm_per_head = self.qk_norm is not None and self.qk_norm.get("per", "projection") == "head"
+        if self.qk_norm is not None and self.qk_norm.get("per", "projection") not in ("head", "projection"):
+            raise ValueError(f"a query/key norm per {self.qk_norm['per']!r}; known: head, projection")
+        if self.conv is not None and (self.norm_per_head or self.value_mix):
+            raise ValueError("behind a convolution queries and keys are normed over the whole projection and values stay unmixed")
+        # what the kernels for equal widths and plain windows do not know
+        self.general = bool(not self.plain_softmax or self.keep_first or self.bias_names or self.value_mix or self.norm_per_head)
         self.q_norm_w = self.k_norm_w = None
 
     @property
     def prepared(self) -> bool:
-        """The step's rows pass the convolution and / or the whole-projection norm on their way into the cache."""
-        return self.conv is not None or self.qk_norm is not None
+        """The step's rows pass a convolution, biases, a norm or a mixing of values on their way into the cache."""
+        return self.conv is not None or self.qk_norm is not None or self.general
 
     def tensor_specs(self):
         specs, seen = [], set()
@@ -136,8 +173,12 @@ class Attention(Mixer):
         if self.conv is not None:
             specs += self.conv.tensor_specs()
         if self.qk_norm is not None:
-            specs += [TensorSpec(self.qk_norm["q_name"], (self.n_heads * self.head_dim,), init="norm_weight"),
-                      TensorSpec(self.qk_norm["k_name"], (self.n_kv_heads * self.head_dim,), init="norm_weight")]
+            heads = (1, 1) if self.norm_per_head else (self.n_heads, self.n_kv_heads)
+            specs += [TensorSpec(self.qk_norm[n], (h * self.head_dim,), init="norm_weight") for n, h in zip(("q_name", "k_name"), heads)]
+        widths = dict(zip(("q_name", "k_name", "v_name", "o_name"), self.qkv.out_features[:3] + [self.hidden]))
+        specs += [TensorSpec(self.bias_names[n], (w,), init="bias") for n, w in widths.items() if n in self.bias_names]
+        if self.value_mix is not None:        # the first layer's share is in the file and enters nothing
+            specs.append(TensorSpec(self.value_mix["share_name"], (), init="share", optional=bool(self.value_mix["first"])))
         return specs
 
     def bind(self, tensors, dtype, device):
@@ -146,6 +187,13 @@ class Attention(Mixer):
         self.q_only = self.qkv.rows(0, self.n_heads * self.head_dim)
         if self.sink_name is not None:
             self.sink = tensors[self.sink_name].float().contiguous()
+        elif self.sink_value is not None:
+            self.sink = torch.full((self.n_heads,), self.sink_value, dtype=torch.float32, device=device)
+        if self.bias_names:
+            self.in_bias = torch.cat([tensors[self.bias_names[n]].float() for n in ("q_name", "k_name", "v_name")]).contiguous()
+            self.out_bias = tensors[self.bias_names["o_name"]].float().contiguous() if "o_name" in self.bias_names else None
+        if self.value_mix is not None and not self.value_mix["first"]:
+            self.mix_share = float(tensors[self.value_mix["share_name"]].float().cpu())
         if self.conv is not None:
             self.conv.bind(tensors, dtype, device)
         if self.qk_norm is not None:
@@ -178,7 +226,7 @@ class Attention(Mixer):
     def cache_need(self):
         kind = "window" if self.window else "chunk" if self.chunk else "full"
         return CacheNeed(kind, self.n_kv_heads, self.head_dim, self.window or self.chunk,
-                         v_dim=None if self.v_dim == self.head_dim else self.v_dim)
+                         v_dim=None if self.v_dim == self.head_dim else self.v_dim, keep=self.keep_first)
 
     @property
     def own_store(self) -> bool:
@@ -194,47 +242,22 @@ class Attention(Mixer):
     def takes_folded(self, ctx, rows: int) -> bool:
         """The q|k|v product can scale its own output rows: in a decode step of few rows, and in a long
         prompt step (the tensor-core product, with or without the rotation in its epilogue)."""
-        if self.prepared or self.gate_name is not None or not self.plain_softmax:
+        if self.prepared or self.gate_name is not None:
             return False
         path = self.qkv.fold_path(ctx, rows, ctx.dtype)
         return path is not None and self.q_only.fold_path(ctx, rows, ctx.dtype) == path and (ctx.is_decode or path == "tiles")
 
     def can_fold(self, ctx, rows: int) -> bool:
         """The output product can finish the sublayer: add to the residual stream and prepare the next norm."""
+        if self.out_bias is not None:
+            return False
         path = self.out.fold_path(ctx, rows, ctx.dtype, finishing=True)
         return path is not None and (ctx.is_decode or path == "tiles")
 
     def _attend(self, qkv, x, ctx, kpages, vpages, block_table, fast_decode, fusion, writes):
         """The step's queries (the leading columns of `qkv`) over the cache -> [T, n_heads * v_dim]."""
         attn = torch.empty((x.shape[0], self.n_heads * self.v_dim), dtype=x.dtype, device=x.device)
-        if not self.plain_softmax:
-            k = ctx.kernels
-            if not qkv.is_contiguous():
-                qkv = qkv.contiguous()
-            dec = ctx.kernels.decode if x.dtype == torch.bfloat16 else None
-            if (ctx.is_decode and dec is not None and self.head_dim in (64, 128)
-                    and dec.uses_tensor_cores(ctx.n_seqs, self.n_heads, self.n_kv_heads, self.head_dim)):
-                # the decode kernel that puts a group's query heads on the tensor cores knows the cap and the sink
-                n_split = ctx.decode_splits(self.n_heads, self.n_kv_heads, self.head_dim)
-                scratch = torch.empty((ctx.n_seqs * self.n_heads * n_split * (self.head_dim + 2),), dtype=torch.float32,
-                                      device=x.device)
-                dec.attn_decode_capped(qkv, attn, ctx.seq_pos0, block_table, kpages, vpages, scratch,
-                                       ctx.engine.tickets(ctx.n_seqs * self.n_kv_heads), ctx.n_seqs, self.n_heads, self.n_kv_heads,
-                                       self.head_dim, self.span, self.scale, n_split, self.softcap, self.sink)
-            elif not ctx.is_decode and x.dtype == torch.bfloat16 and self.head_dim in PrefillAttentionTC.HEAD_DIMS:
-                ctx.kernels.prefill_attention_tc.attn(qkv, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages,
-                                                      ctx.n_seqs, ctx.max_new, self.n_heads, self.n_kv_heads, self.head_dim,
-                                                      self.span, self.scale, ctx.err_flag, self.softcap, self.sink)
-            elif ctx.is_decode and k.attn_decode_split_takes(self.head_dim, qkv.stride(0)):
-                n_split = k.attn_decode_splits(ctx.n_seqs, self.n_heads, self.n_kv_heads, ctx.max_pages, ctx.engine.sm_count)
-                part = torch.empty((ctx.n_seqs * self.n_heads * n_split * (self.head_dim + 2),), dtype=torch.float32,
-                                   device=x.device) if n_split > 1 else None
-                k.attn_decode_split(qkv, attn, ctx.seq_pos0, block_table, kpages, vpages, part, ctx.n_seqs, self.n_heads,
-                                    self.n_kv_heads, self.head_dim, self.span, self.scale, n_split, self.softcap, self.sink)
-            else:
-                k.attn_paged(qkv, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new,
-                             self.n_heads, self.n_kv_heads, self.head_dim, self.span, self.scale, self.softcap, self.sink)
-        elif self.other_widths:
+        if self.other_widths:
             ctx.kernels.seq.attn_wide_value(qkv, attn, ctx.tok_pos, ctx.tok_seq, block_table, kpages, vpages, self.n_heads,
                                             self.n_kv_heads, self.head_dim, self.v_dim, self.span, self.scale)
         elif fast_decode:
@@ -266,12 +289,59 @@ class Attention(Mixer):
                                    ctx.max_new, self.n_heads, self.n_kv_heads, self.head_dim, self.span, self.scale)
         return attn
 
-    def _forward_prepared(self, x, ctx, writes, state, kpages, vpages, block_table, fold):
-        """The path of a layer with a convolution, a whole-projection norm or a gate: one product for queries, keys,
-        values and gate logits; convolution (float32 out); norm, rotation and cache write in one kernel; attention;
-        gate; output product."""
+    def _attend_general(self, q, gate, ctx, unit, kpages, vpages, block_table):
+        """The step's queries [T, n_heads * head_dim] over the cache, with everything `general` stands for; the output
+        [T, n_heads * v_dim] has been multiplied by the sigmoid of `gate` (logits per element, or None)."""
+        T, H, G, hd, vd, k = q.shape[0], self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, ctx.kernels
+        attn = torch.empty((T, H * vd), dtype=q.dtype, device=q.device)
+        if not q.is_contiguous():
+            q = q.contiguous()
+        bf16 = q.dtype == torch.bfloat16
+        options = dict(softcap=self.softcap, sink=self.sink, keep=self.keep_first)
+        fused_gate = gate if gate is not None and bf16 and gate_aligned(gate) else None
+        pages = ctx.pages_seen(unit) if ctx.is_decode else 0
+        if ctx.is_decode and bf16 and DecodeKernels.general_takes(hd, vd):
+            n_split = DecodeKernels.general_splits(ctx.n_seqs, G, hd, vd, pages, ctx.engine.sm_count)
+            scratch = torch.empty((ctx.n_seqs * H * n_split * (vd + 2),), dtype=torch.float32, device=q.device)
+            k.decode.attn_decode_general(q, attn, ctx.seq_pos0, block_table, kpages, vpages, scratch, ctx.engine.tickets(ctx.n_seqs * G),
+                                         ctx.n_seqs, H, G, hd, vd, self.span, self.scale, n_split, gate=fused_gate, **options)
+        elif not ctx.is_decode and bf16 and hd == vd and hd in PrefillAttentionTC.HEAD_DIMS:
+            k.prefill_attention_tc.attn(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, H, G,
+                                        hd, self.span, self.scale, ctx.err_flag, gate=fused_gate, **options)
+        elif not ctx.is_decode and bf16 and PrefillAttentionMMA.takes(hd, vd):
+            k.prefill_attention_mma.attn(q, hd, attn, vd, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs,
+                                         ctx.max_new, H, G, hd, vd, self.span, self.scale, gate=fused_gate, **options)
+        else:
+            fused_gate = None
+            if ctx.is_decode and k.attn_decode_split_takes(hd, q.stride(0), vd):
+                n_split = k.attn_decode_splits(ctx.n_seqs, H, G, pages, ctx.engine.sm_count)
+                part = torch.empty((ctx.n_seqs * H * n_split * (vd + 2),), dtype=torch.float32, device=q.device) if n_split > 1 else None
+                k.attn_decode_split(q, attn, ctx.seq_pos0, block_table, kpages, vpages, part, ctx.n_seqs, H, G, hd, self.span, self.scale,
+                                    n_split, v_dim=vd, **options)
+            else:
+                k.attn_paged(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, H, G, hd,
+                             self.span, self.scale, v_dim=vd, **options)
+        if gate is not None and fused_gate is None:
+            k.gate.head_gate(attn, gate, H * vd, 1)           # "heads" of one column each
+        return attn
+
+    def _value_mix(self, ctx, rows, device):
+        """What the store kernel does with the step's values: (buffer of the group's first layer, None there, else the share)."""
+        if self.value_mix is None:
+            return None
+        key = ("value_mix", self.value_mix.get("group"))
+        if self.value_mix["first"]:
+            ctx.scratch[key] = torch.empty((rows, self.n_kv_heads * self.v_dim), dtype=ctx.dtype, device=device)
+            return ctx.scratch[key], None
+        return ctx.scratch[key], self.mix_share
+
+    def _forward_prepared(self, x, ctx, unit, writes, state, kpages, vpages, block_table, fold):
+        """The path of a layer with a convolution, biases, a query/key norm, mixed values, a gate or anything else that is
+        `general`: one product for queries, keys, values and gate logits; convolution (float32 out); biases, norm, rotation,
+        mixing and cache write in one kernel; attention (with the gate per element where the kernel takes it); gate;
+        output product."""
         if not writes:
-            raise ValueError("a layer with a convolution, a query/key norm or a gate fills its own cache unit")
+            raise ValueError("a layer with a convolution, biases, a query/key norm, a sink or a gate fills its own cache unit")
         T = x.shape[0]
         qw, kw, vw = self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim, self.n_kv_heads * self.v_dim
         y = self.qkv.forward(x, ctx)
@@ -292,18 +362,24 @@ class Attention(Mixer):
                                  self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, rot, interleaved, self.q_norm_w,
                                  self.k_norm_w, eps)
         else:
-            k.qk_norm_store(c, q, ctx.tok_pos, ctx.tok_seq, block_table, table, kpages, vpages, self.n_heads,
-                            self.n_kv_heads, self.head_dim, self.v_dim, rot, interleaved, self.q_norm_w, self.k_norm_w, eps)
-        fast_decode = (ctx.is_decode and x.dtype == torch.bfloat16 and self.head_dim in DecodeKernels.HEAD_DIMS
-                       and not self.other_widths)
-        attn = self._attend(q, x, ctx, kpages, vpages, block_table, fast_decode, None, writes)
-        if self.gate_name is not None and self.gate_per == "head":
-            ctx.kernels.gate.head_gate(attn, y[:, qw + kw + vw:], self.n_heads, self.v_dim)
-        elif self.gate_name is not None:            # a logit per element: "heads" of one column each
-            ctx.kernels.gate.head_gate(attn, y[:, qw + kw + vw:], self.n_heads * self.v_dim, 1)
+            k.qk_norm_store(c, q, ctx.tok_pos, ctx.tok_seq, block_table, table, kpages, vpages, self.n_heads, self.n_kv_heads,
+                            self.head_dim, self.v_dim, rot, interleaved, self.q_norm_w, self.k_norm_w, eps, bias=self.in_bias,
+                            per_head=self.norm_per_head, value_mix=self._value_mix(ctx, T, x.device))
+        gate = y[:, qw + kw + vw:] if self.gate_name is not None else None
+        if self.general:
+            attn = self._attend_general(q, gate if self.gate_per == "element" else None, ctx, unit, kpages, vpages, block_table)
+        else:
+            fast_decode = (ctx.is_decode and x.dtype == torch.bfloat16 and self.head_dim in DecodeKernels.HEAD_DIMS
+                           and not self.other_widths)
+            attn = self._attend(q, x, ctx, kpages, vpages, block_table, fast_decode, None, writes)
+            if gate is not None and self.gate_per == "element":
+                k.head_gate(attn, gate, self.n_heads * self.v_dim, 1)
+        if gate is not None and self.gate_per == "head":
+            k.head_gate(attn, gate, self.n_heads, self.v_dim)
         if fold is not None:
             return self.out.forward_folded(attn, ctx, fold=fold)
-        return self.out.forward(attn, ctx, partials_ok=True)
+        out = self.out.forward(attn, ctx, partials_ok=True)
+        return WithRowVector(out, self.out_bias) if self.out_bias is not None else out
 
     def forward(self, x, ctx, unit, writes, fold=None, state=None):
         if isinstance(x, Folded):
@@ -311,8 +387,8 @@ class Attention(Mixer):
         else:
             folded = None
         kpages, vpages, block_table = ctx.unit_kv(unit)
-        if self.prepared or self.gate_name is not None or not self.plain_softmax:
-            return self._forward_prepared(x, ctx, writes, state, kpages, vpages, block_table, fold)
+        if self.prepared or self.gate_name is not None:
+            return self._forward_prepared(x, ctx, unit, writes, state, kpages, vpages, block_table, fold)
         fast_decode = ctx.is_decode and x.dtype == torch.bfloat16 and self.head_dim in DecodeKernels.HEAD_DIMS
         rotation = self.position.rotation() if self.position is not None else None
         tc = ctx.kernels.tensor_core if x.dtype == torch.bfloat16 else None

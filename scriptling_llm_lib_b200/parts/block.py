@@ -317,7 +317,57 @@ class ParallelInputBlock(Block):
         return self.stream_input.forward(residual, pending, ctx)
 
 
+class PostNormBlock(Block):
+    """x += norm(mixer(x)); then, where the layer has a feed-forward, x += norm(feed_forward(x)): the sublayers read the
+    stream itself, and the norms stand behind them. Roles: `mixer`, `mixer_norm`, and both or neither of `feed_forward`,
+    `feed_forward_norm`. A norm behind a sublayer does not run by itself: the output goes on as the addend the norm makes
+    of it (`addend(y)`, e.g. `rmsnorm`), and the next reader of the stream (this layer's feed-forward, the next layer's
+    mixer, the model's last norm) norms it, adds it and takes its own view of the stream in one pass. That view is the
+    stream rounded to the engine's dtype; in a 32-bit engine the stream itself."""
+
+    def __init__(self, spec: LayerSpec):
+        self.mixer = MIXERS.build(_role(spec, "mixer"))
+        self.mixer_norm = NORMS.build(_role(spec, "mixer_norm"))
+        has = [r in spec.parts for r in ("feed_forward", "feed_forward_norm")]
+        if has[0] != has[1]:
+            raise ValueError("a layer has a feed-forward and its norm, or neither")
+        self.feed_forward = FEED_FORWARDS.build(spec.parts["feed_forward"]) if has[0] else None
+        self.feed_forward_norm = NORMS.build(spec.parts["feed_forward_norm"]) if has[1] else None
+        for norm in (self.mixer_norm, self.feed_forward_norm):
+            if norm is not None and not hasattr(norm, "addend"):
+                raise ValueError(f"{type(norm).__name__} cannot stand behind a sublayer")
+
+    def parts(self):
+        out = [self.mixer, self.mixer_norm]
+        if self.feed_forward is not None:
+            out += [self.feed_forward, self.feed_forward_norm]
+        return out
+
+    @staticmethod
+    def _view(residual, delta, ctx):
+        from .norm import take_into_stream
+        import torch
+        if ctx.dtype == torch.float32:
+            take_into_stream(residual, delta, ctx)
+            return residual
+        xb = torch.empty(residual.shape, dtype=ctx.dtype, device=residual.device)
+        take_into_stream(residual, delta, ctx, xb)
+        return xb
+
+    def forward(self, residual, delta, ctx, unit, writes):
+        h = self._view(residual, delta, ctx)
+        if self.state_need() is not None:
+            a = self.mixer.forward(h, ctx, unit, writes, state=ctx.unit_state(unit))
+        else:
+            a = self.mixer.forward(h, ctx, unit, writes)
+        a = self.mixer_norm.addend(a)
+        if self.feed_forward is None:
+            return a
+        return self.feed_forward_norm.addend(self.feed_forward.forward(self._view(residual, a, ctx), ctx))
+
+
 ARRANGEMENTS.register("pre_norm", PreNormBlock)
+ARRANGEMENTS.register("post_norm", PostNormBlock)
 ARRANGEMENTS.register("parallel_input", ParallelInputBlock)
 ARRANGEMENTS.register("pre_norm_input", PreNormInputBlock)
 ARRANGEMENTS.register("sandwich_norm", SandwichNormBlock)

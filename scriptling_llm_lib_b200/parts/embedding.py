@@ -38,6 +38,34 @@ class TokenEmbedding(Embedding):
         return out
 
 
+class SinusoidEmbedding(TokenEmbedding):
+    """x = E[token] + s(p): at position p of its sequence a token takes a fixed vector (absent in the reference),
+    s_2i = sin(p / base^(2i / width)) and s_2i+1 = cos of the same angle. Angles are made on the host in float64, as
+    (sin, cos) of the positions 0, 64, 128, ... and of 0 .. 63; the kernel puts position 64 a + b together from the two."""
+    STRIDE = 64
+
+    def __init__(self, vocab: int, width: int, name: str, base: float = 10000.0):
+        super().__init__(vocab, width, name)
+        self.base = float(base)
+        self.coarse = self.fine = None
+
+    def prepare(self, max_positions, device):
+        pairs = (self.width + 1) // 2
+        freq = torch.pow(torch.tensor(self.base, dtype=torch.float64), -2.0 * torch.arange(pairs, dtype=torch.float64) / self.width)
+
+        def table(positions):
+            angle = positions.to(torch.float64)[:, None] * freq[None, :]
+            return torch.stack([torch.sin(angle), torch.cos(angle)], dim=-1).to(torch.float32).to(device).contiguous()
+        self.coarse = table(torch.arange(-(-max_positions // self.STRIDE)) * self.STRIDE)
+        self.fine = table(torch.arange(self.STRIDE))
+
+    def forward(self, ids, ctx):
+        out = torch.empty((ids.shape[0], self.width), dtype=torch.float32, device=ids.device)
+        k = ctx.kernels if self.table.dtype == ctx.dtype else ctx.kernels_f32
+        k.embed_rows_sinusoid(ids, ctx.tok_pos, self.table, self.coarse, self.fine, out, ctx.err_flag)
+        return out
+
+
 class PairHashEmbedding(Embedding):
     """x = E[token] + P[r]: a second table P [buckets + 1, width] is looked up by the pair (previous token, token),
     r = (previous * mul_prev + token * mul_cur) mod buckets, and by its last row, r = buckets, for a sequence's first token
@@ -110,6 +138,7 @@ class OutputHead(Head):
 
 
 EMBEDDINGS.register("token_embedding", TokenEmbedding)
+EMBEDDINGS.register("sinusoid_embedding", SinusoidEmbedding)
 EMBEDDINGS.register("pair_hash_embedding", PairHashEmbedding)
 HEADS.register("linear_head", OutputHead)
 

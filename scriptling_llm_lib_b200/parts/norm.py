@@ -1,7 +1,7 @@
 """RMSNorm fused with the residual sum that precedes it.
 
-y = (v / sqrt(mean(v^2) + eps)) * w with v = residual + delta; weight used as is, no bias, no mean
-subtraction (float32_ops.go:159-172). The sum of squares, the division and the residual sum are
+y = (v / sqrt(mean(v^2) + eps)) * w with v = residual + delta; weight used as is (or, `around_zero`, stored as its
+deviation from one), no bias, no mean subtraction (float32_ops.go:159-172). The sum of squares, the division and the residual sum are
 float32 whatever the engine's dtype.
 """
 from __future__ import annotations
@@ -18,20 +18,30 @@ from .base import NORMS, Folded, Norm
 class RMSNorm(Norm):
     graph_safe = True
 
-    def __init__(self, width: int, eps: float, weight_name: str):
-        self.width, self.eps, self.weight_name = width, float(eps), weight_name
+    def __init__(self, width: int, eps: float, weight_name: str, around_zero: bool = False):
+        self.width, self.eps, self.weight_name, self.around_zero = width, float(eps), weight_name, bool(around_zero)
         self.weight = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.weight_name, (self.width,), init="norm_weight")]
+        return [TensorSpec(self.weight_name, (self.width,), init="norm_shift" if self.around_zero else "norm_weight")]
 
     def bind(self, tensors, dtype, device):
         self.weight = tensors[self.weight_name]
+        if self.around_zero:
+            self.weight = self.weight.float() + 1.0
         self.weight_f32 = self.weight if self.weight.dtype == torch.float32 else self.weight.float()
         self._fold_memo = {}
 
     def fold_terms(self):
         return self.weight_f32, self.eps
+
+    def addend(self, y):
+        """A sublayer's output `y` (a tensor in either form, or one with the bias of its last product, `WithRowVector`) as
+        the addend that passes this norm on its way into the stream: the norm stands behind the sublayer."""
+        bias = None
+        if isinstance(y, WithRowVector):
+            y, bias = y.inner, y.vector
+        return RmsNormedAddend(y, self.weight_f32, self.eps, bias)
 
     def forward(self, residual, delta, ctx, rows=None):
         if isinstance(delta, Folded):          # the product before this norm has done its work already
@@ -39,8 +49,12 @@ class RMSNorm(Norm):
         n = residual.shape[0] if rows is None else rows.shape[0]
         y = torch.empty((n, self.width), dtype=ctx.dtype, device=residual.device)
         if isinstance(delta, RmsNormedAddend):  # the addend's own norm, the sum and this norm in one pass
-            ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, norm=(self.weight, self.eps, y), rows=rows)
+            ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, norm=(self.weight, self.eps, y), rows=rows,
+                                            y_bias=delta.bias)
             return y
+        if isinstance(delta, WithRowVector):
+            take_into_stream(residual, delta, ctx)
+            delta = None
         ctx.kernels.add_rmsnorm(residual, delta, rows, self.weight, y, self.eps)
         return y
 
@@ -48,14 +62,16 @@ class RMSNorm(Norm):
 @dataclass
 class RmsNormedAddend:
     """An addend that joins the residual stream divided by its own root mean square: x += y / sqrt(mean(y^2) + eps) * weight.
-    `y` is [T, width] (float32 or the engine's dtype) or float32 [P, T, width] partial sums, `weight` float32. The RMS norm
-    that reads the stream next does both in one pass; `apply` does the sum by itself for a reader that is none."""
+    `y` is [T, width] (float32 or the engine's dtype) or float32 [P, T, width] partial sums, `weight` float32; `bias`
+    (float32 [width], or None) is added to y before its norm. The RMS norm that reads the stream next does both in one
+    pass; `apply` does the sum by itself for a reader that is none."""
     y: Any
     weight: Any
     eps: float
+    bias: Any = None
 
     def apply(self, residual, ctx) -> None:
-        ctx.kernels.gate.add_rms_normed(residual, self.y, self.weight, self.eps)
+        ctx.kernels.gate.add_rms_normed(residual, self.y, self.weight, self.eps, y_bias=self.bias)
 
 
 class WeightedNorm(Norm):
@@ -109,8 +125,8 @@ def take_into_stream(residual, delta, ctx, xb=None) -> None:
     if isinstance(delta, WithRowVector):
         delta, vec = delta.inner, delta.vector
     if isinstance(delta, RmsNormedAddend):
-        ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, vec=vec)
-        delta, vec = None, None
+        ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, vec=vec, y_bias=delta.bias, copy=xb)
+        delta, vec, xb = None, None, None
     if isinstance(delta, NormedAddend):
         raise ValueError("an addend that still has to pass a norm of its own is taken in by the norm that reads the stream next")
     addends = [] if delta is None else list(delta) if isinstance(delta, (list, tuple)) else [delta]
@@ -164,7 +180,7 @@ class DynamicTanh(Norm):
         n = residual.shape[0] if rows is None else rows.shape[0]
         if isinstance(delta, RmsNormedAddend):
             y = torch.empty((n, self.width), dtype=ctx.dtype, device=residual.device)
-            ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, rows=rows, vec=vec,
+            ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, rows=rows, vec=vec, y_bias=delta.bias,
                                             dyt=(self.weight, self.bias, self.alpha, y))
             return y
         if isinstance(delta, (list, tuple)) or vec is not None:

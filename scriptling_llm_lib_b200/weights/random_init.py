@@ -51,6 +51,8 @@ INIT_LAWS: dict[str, Normal | UniformInteger] = {
     "matrix": Normal(0.0, MATRIX_STD),
     "norm_weight": Normal(1.0, MATRIX_STD),
     "integer_table": UniformInteger(2 ** 15),
+    "norm_shift": Normal(0.0, 0.1),         # a norm's weight stored as its deviation from one
+    "share": Normal(0.4, 0.1),              # how much of another layer's values a layer takes in
     "conv_filter": Normal(0.0, 0.3),        # the taps of a short convolution over time
     "bias": Normal(0.0, 0.1),
     "log_rate": Normal(0.0, 0.5),           # logarithms of decay rates (a recurrence's A_log, lambda)
