@@ -556,8 +556,34 @@ def tufazen_config(z):
             "token_side": {"dim": z["side"]}, "vocab": DESIGN_VOCAB, "width": z["width"]}
 
 
+# The Fopezen decoder (grouped-query attention in two forms with biases, query/key norms, a window that keeps the sequence's
+# first positions, mixed values, in one of them a sink and an elementwise gate; square-of-relu feed-forwards; norms behind the
+# sublayers; sines and cosines of the position on the embedding) at layer sizes that resemble real models of its kinds: heads of
+# 128, windows of 1024 with 16 positions kept, a wider window in every fourth layer's `attention_2`. w2048-v64 has values half
+# as wide as the keys. The Llama decoder beside it has the same width, depth, heads and window; its gated feed-forward has three
+# matrices, so two thirds of the width give it the same FLOPs.
+FOPEZEN_SIZES = {
+    "w1024": dict(width=1024, heads=8, kv_heads=2, dim=128, vdim=128, window=1024, keep=16, dense_ff=4096, layers=4),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, window=1024, keep=16, dense_ff=8192, layers=4),
+    "w2048-v64": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=64, window=1024, keep=16, dense_ff=8192, layers=4),
+}
+for _z in FOPEZEN_SIZES.values():
+    _z.update(ff=-(-2 * _z["dense_ff"] // 3 // 256) * 256, groups=1)
+
+
+def fopezen_config(z):
+    def layer(i):
+        wide = i % 4 == 0
+        return {"type": "attention_2" if wide else "attention", "mlp": {"ff": z["dense_ff"], "kind": "dense"}, "mixer": {
+            "dim": z["dim"], "heads": z["heads"], "kv_heads": z["kv_heads"], "scale": z["dim"] ** -0.5, "v_mix": True, "vdim": z["vdim"],
+            "mask": {"keep_first": z["keep"], "size": z["window"] * (2 if wide else 1)}}}
+    return {"architecture": "Fopezen", "layers": [layer(i) for i in range(z["layers"])], "norm": {"eps": 1e-6}, "vocab": DESIGN_VOCAB,
+            "width": z["width"]}
+
+
 DESIGNS = {"sozilix": (DESIGN_SIZES, sozilix_config, 3), "muvorax": (MUVORAX_SIZES, muvorax_config, 6),
-           "belasun": (BELASUN_SIZES, belasun_config, 4), "tufazen": (TUFAZEN_SIZES, tufazen_config, 6)}
+           "belasun": (BELASUN_SIZES, belasun_config, 4), "tufazen": (TUFAZEN_SIZES, tufazen_config, 6),
+           "fopezen": (FOPEZEN_SIZES, fopezen_config, 4)}
 
 
 def llama_like(z, max_positions, layers_per_group=3):
@@ -1310,6 +1336,154 @@ def kernel_alone(args):
     return 0
 
 
+def fopezen_kernels_alone(args):
+    """What the Fopezen decoder added to the kernels, each alone at FOPEZEN_SIZES[--design-sizes or w2048] beside its like on
+    the same rows: attention over a window with kept positions, a sink and a gate beside the same window without (and, where
+    values are narrower than keys, beside the kernel for equal widths), the store kernel with biases, query/key norm and mixed
+    values beside the rotation-and-store kernel, the normed addend with a bias and the stream's copy beside the sum with an RMS
+    norm, the embedding with positions beside the plain one, the product with the square of relu beside the plain product. A
+    prompt of --prefill-tokens rows and a decode step of --batch rows at --context; a JSON line each (CUDA events around a
+    captured run of launches; inputs rotate through more than L2 holds where they are small)."""
+    import torch
+    from scriptling_llm_lib_b200.csrc.bindings import DecodeKernels, KernelSet
+    pk = peaks()
+    z = FOPEZEN_SIZES[(args.design_sizes or "w2048").split(",")[0]]
+    dt, dev, esz = torch.bfloat16, "cuda", 2
+    ks = KernelSet(dt)
+    W, H, G, D, V, F, window, keep = (z[n] for n in ("width", "heads", "kv_heads", "dim", "vdim", "dense_ff", "window", "keep"))
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+
+    def timed(launch, n_sets, reps=8):
+        torch.cuda.synchronize()
+        side = torch.cuda.Stream()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.stream(side):
+            for i in range(2):
+                launch(i % n_sets)
+            torch.cuda.synchronize()
+            with torch.cuda.graph(graph, stream=side):
+                for i in range(max(reps, n_sets)):
+                    launch(i % n_sets)
+        for _ in range(3):
+            graph.replay()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        for _ in range(5):
+            graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / (5 * max(reps, n_sets)) * 1e3
+
+    def report(name, rows, us, nbytes=None, flops=None, like=None):
+        rec = {"kernel": name, "rows": rows, "us": round(us, 2)}
+        if like is not None:
+            rec["like"] = like
+        if nbytes is not None:
+            rec.update(gbs=round(nbytes / us / 1e3, 1), of_hbm=round(nbytes / us / 1e3 / pk["hbm_gbs"], 3))
+        if flops is not None:
+            rec.update(tflops=round(flops / us / 1e6, 1), of_bf16=round(flops / us / 1e6 / pk["bf16_tflops"], 3))
+        print(json.dumps(rec), flush=True)
+
+    err = torch.zeros(1, dtype=torch.int32, device=dev)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rand = lambda *shape: torch.randn(*shape, device=dev).to(dt)
+    for label in ("prompt", "decode"):
+        T, B, ctxlen = (args.prefill_tokens, 1, args.prefill_tokens) if label == "prompt" else (args.batch, args.batch, args.context)
+        pages = -(-ctxlen // 64)
+        seq_start, pos0 = (i32([0, T]), i32([0])) if B == 1 and T > 1 else (torch.arange(B + 1, dtype=torch.int32, device=dev), i32([ctxlen - 1] * B))
+        tok_pos = torch.arange(T, dtype=torch.int32, device=dev) if label == "prompt" else pos0.clone()
+        tok_seq = torch.zeros(T, dtype=torch.int32, device=dev) if label == "prompt" else torch.arange(B, dtype=torch.int32, device=dev)
+        table = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages).contiguous()
+        n_sets = 4 if T > 64 else 24
+        # caches in sets that rotate through more than L2 holds
+        kv_sets = 1 if label == "prompt" else max(1, -(-200_000_000 // (B * min(ctxlen, window + 64) * G * (D + V) * esz)))
+        kv_sets = min(kv_sets, 12)
+        kp, vp = [rand(B * pages + 1, G, 64, D) for _ in range(kv_sets)], [rand(B * pages + 1, G, 64, V) for _ in range(kv_sets)]
+        q, o, gates = rand(T, H * D), torch.empty(T, H * V, dtype=dt, device=dev), rand(T, H * V)
+        sink = torch.zeros(H, device=dev)
+        full = dict(sink=sink, keep=keep, gate=gates)
+        seen = sum(min(i + 1, window) for i in range(T)) if label == "prompt" else B * min(ctxlen, window)
+        what = f"{H}/{G} heads of {D}/{V}, window {window}"
+        if label == "prompt":
+            flops, tc, mma = 2 * H * (D + V) * seen, ks.prefill_attention_tc, ks.prefill_attention_mma
+            run_mma = lambda opts: timed(lambda i: mma.attn(q, D, o, V, seq_start, pos0, table, kp[0], vp[0], 1, T, H, G, D, V, window,
+                                                            D ** -0.5, **opts), 1)
+            if D == V and D in tc.HEAD_DIMS:
+                run_tc = lambda opts: timed(lambda i: tc.attn(q, o, seq_start, pos0, table, kp[0], vp[0], 1, T, H, G, D, window, D ** -0.5,
+                                                              err, **opts), 1)
+                report(f"attn_prefill (tcgen05) {what}, {keep} kept, sink, gate ({label})", T, run_tc(full), flops=flops)
+                report(f"attn_prefill (tcgen05) {what}, plain ({label})", T, run_tc({}), flops=flops, like="kept, sink, gate")
+            else:
+                report(f"attn_prefill_mma {what}, {keep} kept, sink, gate ({label})", T, run_mma(full), flops=flops)
+                vq, oq = rand(B * pages + 1, G, 64, D), torch.empty(T, H * D, dtype=dt, device=dev)
+                us = timed(lambda i: tc.attn(q, oq, seq_start, pos0, table, kp[0], vq, 1, T, H, G, D, window, D ** -0.5, err), 1)
+                report(f"attn_prefill (tcgen05) {H}/{G} heads of {D}, window {window}, plain ({label})", T, us, flops=4 * H * D * seen,
+                       like="attn_prefill_mma")
+        else:
+            seen_pages = min(pages, (window + 126) // 64 + -(-keep // 64))
+            n_split = DecodeKernels.general_splits(B, G, D, V, seen_pages, sms)
+            scratch, tickets = torch.empty(B * H * n_split * (V + 2), device=dev), torch.zeros(B * G, dtype=torch.int32, device=dev)
+            us = timed(lambda i: ks.decode.attn_decode_general(q, o, pos0, table, kp[i], vp[i], scratch, tickets, B, H, G, D, V, window,
+                                                               D ** -0.5, n_split, **full), kv_sets)
+            report(f"attn_decode_general {what}, {keep} kept, sink, gate, {n_split} splits ({label})", T, us,
+                   nbytes=B * min(ctxlen, window + keep) * G * (D + V) * esz)
+            oq = torch.empty(T, H * D, dtype=dt, device=dev)
+            vq = vp if V == D else [rand(B * pages + 1, G, 64, D) for _ in range(kv_sets)]
+            ns = ks.decode.attention_splits(B, H, G, D, pages, sms)
+            sc2 = torch.empty(B * H * ns * (D + 2), device=dev)
+            us = timed(lambda i: ks.decode.attn_decode(q, oq, pos0, table, kp[i], vq[i], sc2, B, H, G, D, window, D ** -0.5, ns,
+                                                       tickets=tickets), kv_sets)
+            report(f"attn_decode {H}/{G} heads of {D}, window {window}, plain, {ns} splits ({label})", T, us,
+                   nbytes=B * min(ctxlen, window) * G * 2 * D * esz, like="attn_decode_general")
+        # ---- biases, query/key norm, mixed values, cache write; beside rotation and cache write
+        C, Cg = (H + G) * D + G * V, (H + G) * D + G * V + H * V
+        ys = [rand(T, Cg) for _ in range(n_sets)]
+        bias, qn, kn = torch.randn(C, device=dev), torch.rand(D, device=dev) + 0.5, torch.rand(D, device=dev) + 0.5
+        qw, kw = torch.rand(H * D, device=dev) + 0.5, torch.rand(G * D, device=dev) + 0.5
+        qo, kept = torch.empty(T, H * D, dtype=dt, device=dev), rand(T, G * V)
+        moved = T * (2 * C + G * V) * esz
+        for name, per_head, w, mix in (("norm per head, values mixed", True, (qn, kn), (kept, 0.3)), ("norm over the projection, values kept",
+                                                                                                     False, (qw, kw), (kept, None))):
+            us = timed(lambda i: ks.gate.qk_norm_store(ys[i][:, :C], qo, tok_pos, tok_seq, table, None, kp[0], vp[0], H, G, D, V, 0, False, *w,
+                                                       1e-6, bias=bias, per_head=per_head, value_mix=mix), n_sets)
+            report(f"qk_norm_store, biases, {name} ({label})", T, us, nbytes=moved)
+        if D == V:
+            rows = [rand(T, C) for _ in range(n_sets)]
+            cs = torch.randn(ctxlen + 1, D // 2, 2, device=dev)
+            us = timed(lambda i: ks.rope_kv_write(rows[i], tok_pos, tok_seq, table, cs, kp[0], vp[0], H, G, D, D, False), n_sets)
+            report(f"rope_kv_write ({label})", T, us, nbytes=2 * T * C * esz, like="qk_norm_store")
+        # ---- x += (y + b) / rms(y + b) w and the rounded copy; beside the sum with an RMS norm behind it
+        xs = [torch.randn(T, W, device=dev) for _ in range(n_sets)]
+        y2, out, w1, b1 = [rand(T, W) for _ in range(n_sets)], torch.empty(T, W, dtype=dt, device=dev), torch.randn(W, device=dev), torch.randn(W, device=dev)
+        us = timed(lambda i: ks.gate.add_rms_normed(xs[i], y2[i], w1, 1e-6, y_bias=b1, copy=out), n_sets)
+        report(f"add_rms_normed, bias and copy ({label})", T, us, nbytes=T * W * (8 + 2 * esz))
+        us = timed(lambda i: ks.add_rmsnorm(xs[i], y2[i], None, w1, out, 1e-6), n_sets)
+        report(f"add_rmsnorm ({label})", T, us, nbytes=T * W * (8 + 2 * esz), like="add_rms_normed")
+        # ---- the embedding with sines and cosines, beside the plain one
+        tab = rand(DESIGN_VOCAB, W)
+        tok = torch.randint(0, DESIGN_VOCAB, (T,), dtype=torch.int32, device=dev)
+        coarse, fine = torch.randn(pages + 1, W // 2, 2, device=dev), torch.randn(64, W // 2, 2, device=dev)
+        us = timed(lambda i: ks.embed_rows_sinusoid(tok, tok_pos, tab, coarse, fine, xs[i], err), n_sets)
+        report(f"embed_rows_sinusoid ({label})", T, us, nbytes=T * W * (esz + 4))
+        us = timed(lambda i: ks.embed_rows(tok, tab, xs[i], err), n_sets)
+        report(f"embed_rows ({label})", T, us, nbytes=T * W * (esz + 4), like="embed_rows_sinusoid")
+        # ---- the feed-forward's first product with the square of relu, beside the plain product
+        xin, hid = rand(T, W), torch.empty(T, F, dtype=dt, device=dev)
+        wu = [rand(F, W) * 0.02 for _ in range(1 if T > 64 else 8)]
+        if T > 128:
+            us = timed(lambda i: ks.tensor_core.gemm_act(xin, wu[0], hid, err, "relu_squared"), 1)
+            report(f"up product with relu squared, {F} x {W} ({label})", T, us, flops=2 * T * F * W)
+            us = timed(lambda i: ks.tensor_core.gemm(xin, wu[0], hid, err), 1)
+            report(f"up product, plain, {F} x {W} ({label})", T, us, flops=2 * T * F * W, like="relu squared")
+        else:
+            us = timed(lambda i: (ks.decode.gemm_small_m(xin, wu[i], hid), ks.mix.act_inplace(hid, "relu_squared")), len(wu))
+            report(f"up product and relu squared, {F} x {W} ({label})", T, us, nbytes=F * W * esz)
+            us = timed(lambda i: ks.decode.gemm_small_m(xin, wu[i], hid), len(wu))
+            report(f"up product, plain, {F} x {W} ({label})", T, us, nbytes=F * W * esz, like="relu squared")
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1335,7 +1509,7 @@ def main():
     ap.add_argument("--no-shapes", dest="shapes", action="store_false", help="skip the Llama-3.2-1B and Llama-3.1-8B sizes")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode"],
                     help="run one part only (a small case to profile); the JSON line then holds that part alone")
-    ap.add_argument("--kernel", default=None, choices=["attn_decode", "gemm_small_m", "sequence", "mix", "gate", "tufazen"],
+    ap.add_argument("--kernel", default=None, choices=["attn_decode", "gemm_small_m", "sequence", "mix", "gate", "tufazen", "fopezen"],
                     help="time one decode kernel alone at --shape, --batch (and --context) instead of the model; 'sequence': "
                          "the kernels of the mixers with state at --design-sizes, for a prompt and for a decode step; 'mix': "
                          "the same for the kernels of latent attention, decayed linear attention, the selective scan and "
@@ -1343,7 +1517,9 @@ def main():
                          "the projections, whole-projection norm, gate per head, chunked attention, gated experts, token input); 'tufazen': "
                          "what the Tufazen decoder added (capped attention with sinks, sums of several addends, the normed addend "
                          "before a tanh norm, the pair-table embedding, the gate per element, the router over groups, the dense "
-                         "clamped gate), each beside its like")
+                         "clamped gate), each beside its like; 'fopezen': what the Fopezen decoder added (attention over a window "
+                         "with kept positions, a sink and a gate, biases with query/key norm and mixed values in the store kernel, "
+                         "the normed addend with a bias and a copy, the embedding with positions, the square of relu), likewise")
     ap.add_argument("--design", default=None, choices=sorted(DESIGNS),
                     help="measure this design's prompt step and decoding at a few real layer sizes beside the Llama decoder "
                          "of equal size (--prefill-tokens, --batch, --context, --steps, --dtype, --only apply) instead of the "
@@ -1366,6 +1542,8 @@ def main():
         return mix_kernels_alone(args)
     if args.kernel == "tufazen":
         return tufazen_kernels_alone(args)
+    if args.kernel == "fopezen":
+        return fopezen_kernels_alone(args)
     if args.kernel is not None:
         return kernel_alone(args)
     if args.design is not None:
