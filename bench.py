@@ -1406,20 +1406,13 @@ def fopezen_kernels_alone(args):
         seen = sum(min(i + 1, window) for i in range(T)) if label == "prompt" else B * min(ctxlen, window)
         what = f"{H}/{G} heads of {D}/{V}, window {window}"
         if label == "prompt":
-            flops, tc, mma = 2 * H * (D + V) * seen, ks.prefill_attention_tc, ks.prefill_attention_mma
-            run_mma = lambda opts: timed(lambda i: mma.attn(q, D, o, V, seq_start, pos0, table, kp[0], vp[0], 1, T, H, G, D, V, window,
-                                                            D ** -0.5, **opts), 1)
-            if D == V and D in tc.HEAD_DIMS:
-                run_tc = lambda opts: timed(lambda i: tc.attn(q, o, seq_start, pos0, table, kp[0], vp[0], 1, T, H, G, D, window, D ** -0.5,
-                                                              err, **opts), 1)
-                report(f"attn_prefill (tcgen05) {what}, {keep} kept, sink, gate ({label})", T, run_tc(full), flops=flops)
-                report(f"attn_prefill (tcgen05) {what}, plain ({label})", T, run_tc({}), flops=flops, like="kept, sink, gate")
-            else:
-                report(f"attn_prefill_mma {what}, {keep} kept, sink, gate ({label})", T, run_mma(full), flops=flops)
-                vq, oq = rand(B * pages + 1, G, 64, D), torch.empty(T, H * D, dtype=dt, device=dev)
-                us = timed(lambda i: tc.attn(q, oq, seq_start, pos0, table, kp[0], vq, 1, T, H, G, D, window, D ** -0.5, err), 1)
-                report(f"attn_prefill (tcgen05) {H}/{G} heads of {D}, window {window}, plain ({label})", T, us, flops=4 * H * D * seen,
-                       like="attn_prefill_mma")
+            flops, tc = 2 * H * (D + V) * seen, ks.prefill_attention_tc
+            us = timed(lambda i: tc.attn(q, o, seq_start, pos0, table, kp[0], vp[0], 1, T, H, G, D, window, D ** -0.5, err, v_dim=V, **full), 1)
+            report(f"attn_prefill {what}, {keep} kept, sink, gate ({label})", T, us, flops=flops)
+            vq, oq = vp[0] if V == D else rand(B * pages + 1, G, 64, D), torch.empty(T, H * D, dtype=dt, device=dev)
+            us = timed(lambda i: tc.attn(q, oq, seq_start, pos0, table, kp[0], vq, 1, T, H, G, D, window, D ** -0.5, err), 1)
+            report(f"attn_prefill {H}/{G} heads of {D}, window {window}, plain ({label})", T, us, flops=4 * H * D * seen,
+                   like="kept, sink, gate")
         else:
             seen_pages = min(pages, (window + 126) // 64 + -(-keep // 64))
             n_split = DecodeKernels.general_splits(B, G, D, V, seen_pages, sms)
@@ -1477,7 +1470,7 @@ def fopezen_kernels_alone(args):
             us = timed(lambda i: ks.tensor_core.gemm(xin, wu[0], hid, err), 1)
             report(f"up product, plain, {F} x {W} ({label})", T, us, flops=2 * T * F * W, like="relu squared")
         else:
-            us = timed(lambda i: (ks.decode.gemm_small_m(xin, wu[i], hid), ks.mix.act_inplace(hid, "relu_squared")), len(wu))
+            us = timed(lambda i: ks.decode.gemm_small_m_act(xin, wu[i], hid, "relu_squared"), len(wu))
             report(f"up product and relu squared, {F} x {W} ({label})", T, us, nbytes=F * W * esz)
             us = timed(lambda i: ks.decode.gemm_small_m(xin, wu[i], hid), len(wu))
             report(f"up product, plain, {F} x {W} ({label})", T, us, nbytes=F * W * esz, like="relu squared")

@@ -1,5 +1,5 @@
 // Causal grouped-query attention of a prompt step over the paged cache on tcgen05 tensor cores
-// (bfloat16, head width 64 or 128; a head of 128 is two 64-wide swizzled blocks side by side in
+// (bfloat16; built for keys and values of 64 or 128 dims, narrower heads in multiples of 8; a head of 128 is two 64-wide swizzled blocks side by side in
 // shared memory for Q, K and V alike, and O takes 128 columns of tensor memory).
 //
 // Common to both head widths. A query tile is 128 consecutive queries of one sequence and one
@@ -48,14 +48,14 @@ struct FtArgs {
   const int* seq_pos0;  // [B]
   const int* block_table;
   int max_pages;
-  int H, G, window, keep;
+  int H, G, hd, vd, window, keep;   // hd, vd: the widths used, at most what the kernel is built for
   float scale;
   int* err;
   int n_qt, n_seqs, n_items;   // query tiles per sequence (of the longest), sequences, work items
   int pair_heads;              // pair kernel: 1: an item is heads 2i, 2i+1 on one query tile; 0: query tiles 2i, 2i+1 of one head
   float softcap;               // > 0: a score s (scaled) becomes softcap * tanh(s / softcap) before the softmax
   const float* sink;           // [H] or null: exp(sink[h]) joins head h's denominator, with no key and no value
-  const bf16* gate;            // null, or [T, gate_ld]: output element (h, d) is multiplied by the sigmoid of column h * hd + d
+  const bf16* gate;            // null, or [T, gate_ld]: output element (h, d) is multiplied by the sigmoid of column h * vd + d
   int gate_ld;
 };
 
@@ -106,10 +106,11 @@ __device__ __forceinline__ float ft_tanh(float x) {
 __device__ __forceinline__ uint32_t ft_cap(uint32_t s, float cap_out, float cap_in) {
   return __float_as_uint(cap_out * ft_tanh(__uint_as_float(s) * cap_in));
 }
-// 32 output elements times the sigmoid of their gate logits (16-byte aligned)
-__device__ __forceinline__ void ft_gate(uint32_t (&v)[32], const bf16* g) {
+// the first n of 32 output elements (n a multiple of 8) times the sigmoid of their gate logits (16-byte aligned)
+__device__ __forceinline__ void ft_gate(uint32_t (&v)[32], const bf16* g, int n) {
 #pragma unroll
   for (int c = 0; c < 4; c++) {
+    if (8 * c >= n) break;
     const uint4 w = *(const uint4*)(g + 8 * c);
     const bf16* e = (const bf16*)&w;
 #pragma unroll
@@ -155,6 +156,8 @@ __device__ __forceinline__ void umma_bf16_ta(uint32_t tmem_d, uint32_t tmem_a, u
                ::"r"(tmem_d), "r"(tmem_a), "l"(db), "r"(idesc), "r"(accumulate) : "memory");
 }
 
+// Heads of up to FT_HD dims for keys and values alike, in multiples of 8: TMA fills a box's columns past the storage row with
+// zeros, what a query box holds past its head meets those zeros, and only p.vd columns are written out.
 template <int FT_HD, int FT_STAGES>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -214,7 +217,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         if (!mbar_wait(b_qempty, (I & 1) ^ 1, abort)) break;
         mbar_expect_tx(b_qfull, Q_BYTES);
 #pragma unroll
-        for (int a = 0; a < NA; a++) tma_load_2d(sQ + a * QA, &map_q, it.h * FT_HD + 64 * a, it.row0 + it.r0, b_qfull);
+        for (int a = 0; a < NA; a++) tma_load_2d(sQ + a * QA, &map_q, it.h * p.hd + 64 * a, it.row0 + it.r0, b_qfull);
         I++;
         for (int j = 0; j < it.n_tiles; j++) {
           int s = J % FT_STAGES;
@@ -255,7 +258,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
           for (int k = 0; k < FT_HD / 16; k++)      // 16 dims a step: four steps in each 64-wide block
-            umma_bf16(tmem_base + a * 64, umma_desc_sw128(sQ + (k >> 2) * QA + (k & 3) * 32),
+            if (16 * k < p.hd) umma_bf16(tmem_base + a * 64, umma_desc_sw128(sQ + (k >> 2) * QA + (k & 3) * 32),
                       umma_desc_sw128(sK + s * KV_BYTES + (k >> 2) * KA + (k & 3) * 32), idesc_s, k ? 1u : 0u);
           umma_commit(b_sfull + 8 * a);
           if (j == n_tiles - 1) umma_commit(b_qempty);     // the item's last product that reads Q
@@ -403,14 +406,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       if (p.sink != nullptr) l = (m_ref == -INFINITY) ? 1.f : l + ft_ex2(p.sink[h] * FT_LOG2E - m_ref * sc);
       float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = p.out + (size_t)(row0 + r0 + r) * ((size_t)p.H * FT_HD) + (size_t)h * FT_HD;
+      bf16* dst = p.out + (size_t)(row0 + r0 + r) * ((size_t)p.H * p.vd) + (size_t)h * p.vd;
 #pragma unroll 1
       for (int c0 = 0; c0 < FT_HD; c0 += 32) {
         uint32_t v[32];
         tmem_ld32(t_lane + 128 + c0, v);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (r < nq) {
-          if (p.gate != nullptr) ft_gate(v, p.gate + (size_t)(row0 + r0 + r) * p.gate_ld + (size_t)h * FT_HD + c0);
+          if (p.gate != nullptr) ft_gate(v, p.gate + (size_t)(row0 + r0 + r) * p.gate_ld + (size_t)h * p.vd + c0, p.vd - c0);
 #pragma unroll
           for (int c = 0; c < 4; c++) {
             uint4 w;
@@ -419,7 +422,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             __nv_bfloat162 p2 = __floats2bfloat162_rn(__uint_as_float(v[8 * c + 4]) * inv, __uint_as_float(v[8 * c + 5]) * inv);
             __nv_bfloat162 p3 = __floats2bfloat162_rn(__uint_as_float(v[8 * c + 6]) * inv, __uint_as_float(v[8 * c + 7]) * inv);
             w.x = *(uint32_t*)&p0; w.y = *(uint32_t*)&p1; w.z = *(uint32_t*)&p2; w.w = *(uint32_t*)&p3;
-            *(uint4*)(dst + c0 + 8 * c) = w;
+            if (c0 + 8 * c < p.vd) *(uint4*)(dst + c0 + 8 * c) = w;
           }
         }
       }
@@ -533,23 +536,24 @@ __device__ __forceinline__ void ft_ld64(uint32_t taddr, uint32_t (&s)[64]) {
   tmem_ld32(taddr + 32, *(uint32_t(*)[32])&s[32]);
 }
 
-template <int FT_HD, int FT_STAGES>
+// Keys of up to KD and values of up to VD dims (64 or 128 either, not both 64: that is the kernel above), narrower heads as there.
+template <int KD, int VD, int FT_STAGES>
 __global__ void __launch_bounds__(FP_THREADS, 1)
 attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, FtArgs p, uint32_t smem_bytes) {
-  constexpr uint32_t Q_BYTES = FT_BQ * FT_HD * 2, KV_BYTES = FT_BK * FT_HD * 2;
+  constexpr uint32_t Q_BYTES = FT_BQ * KD * 2, K_BYTES = FT_BK * KD * 2, V_BYTES = FT_BK * VD * 2;
   constexpr uint32_t QA = FT_BQ * 128, KA = FT_BK * 128;       // bytes of one 64-wide block of Q and of a K or V page
-  constexpr int NA = FT_HD / 64;                               // such blocks per head
-  // tensor-memory columns of one tile of the pair (256): a head of 64 has S0 0-63, S1 64-127, O 128-191, P0 192-223,
-  // P1 224-255; a head of 128, whose O takes 128-255, has one S buffer 0-63 and P0 64-95, P1 96-127
-  constexpr int NBUF = FT_HD > 64 ? 1 : 2;       // S buffers; the next tile's S is issued while a tile's softmax runs
-  constexpr uint32_t P_COL0 = FT_HD > 64 ? 64 : 192, P_STEP = 32, SUB_COLS = 256;
+  constexpr int NK = KD / 64, NV = VD / 64;                    // such blocks per key (query) head and per value head
+  // tensor-memory columns of one tile of the pair (256): values of 64 have S0 0-63, S1 64-127, O 128-191, P0 192-223,
+  // P1 224-255; values of 128, whose O takes 128-255, have one S buffer 0-63 and P0 64-95, P1 96-127
+  constexpr int NBUF = VD > 64 ? 1 : 2;          // S buffers; the next tile's S is issued while a tile's softmax runs
+  constexpr uint32_t P_COL0 = VD > 64 ? 64 : 192, P_STEP = 32, SUB_COLS = 256;
   static_assert(FT_STAGES >= 3, "the key/value ring must hold the tile whose S is issued ahead");
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   // [Q of either tile][K stages][V stages][barriers]
-  const uint32_t sQ = smem_u32(smem), sK = sQ + 2 * Q_BYTES, sV = sK + FT_STAGES * KV_BYTES;
-  uint64_t* bars = (uint64_t*)(smem + 2 * Q_BYTES + 2 * FT_STAGES * KV_BYTES);
+  const uint32_t sQ = smem_u32(smem), sK = sQ + 2 * Q_BYTES, sV = sK + FT_STAGES * K_BYTES;
+  uint64_t* bars = (uint64_t*)(smem + 2 * Q_BYTES + FT_STAGES * (K_BYTES + V_BYTES));
   // q_full, q_empty, kv_full[ST], kv_empty[ST], then for either tile of the pair s_full[2], s_empty[2], p_full[2],
   // o_full[2]. The barriers of P and O come in pairs, one for the tiles of each parity, those of S one per
   // buffer: a waiter is then never more than one phase behind.
@@ -608,8 +612,8 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           for (int x = 0; x < 2; x++)
             if (it.sub[x].valid) {
 #pragma unroll
-              for (int a = 0; a < NA; a++)
-                tma_load_2d(sQ + x * Q_BYTES + a * QA, &map_q, it.sub[x].h * FT_HD + 64 * a, it.row0 + it.sub[x].r0, b_qfull);
+              for (int a = 0; a < NK; a++)
+                tma_load_2d(sQ + x * Q_BYTES + a * QA, &map_q, it.sub[x].h * p.hd + 64 * a, it.row0 + it.sub[x].r0, b_qfull);
             }
           I++;
           for (int u = 0; u < it.n_union; u++) {
@@ -617,12 +621,11 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             if (!mbar_wait(b_kvempty + 8 * s, ((JU / FT_STAGES) & 1) ^ 1, abort)) { ok = false; break; }
             int page = bt[fp_union_tile(it, u)];
             int krow = (page * p.G + it.g) * FT_BK;
-            mbar_expect_tx(b_kvfull + 8 * s, 2 * KV_BYTES);
+            mbar_expect_tx(b_kvfull + 8 * s, K_BYTES + V_BYTES);
 #pragma unroll
-            for (int a = 0; a < NA; a++) {
-              tma_load_2d(sK + s * KV_BYTES + a * KA, &map_k, 64 * a, krow, b_kvfull + 8 * s);
-              tma_load_2d(sV + s * KV_BYTES + a * KA, &map_v, 64 * a, krow, b_kvfull + 8 * s);
-            }
+            for (int a = 0; a < NK; a++) tma_load_2d(sK + s * K_BYTES + a * KA, &map_k, 64 * a, krow, b_kvfull + 8 * s);
+#pragma unroll
+            for (int a = 0; a < NV; a++) tma_load_2d(sV + s * V_BYTES + a * KA, &map_v, 64 * a, krow, b_kvfull + 8 * s);
             JU++;
           }
         }
@@ -636,7 +639,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       if (lane == 0) {
         const int x = warp - 1;                    // this thread issues the products of one tile of the pair
         constexpr uint32_t idesc_s = umma_idesc_bf16(FT_BQ, FT_BK);          // S = Q K^T: both K-major
-        constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(FT_BQ, FT_HD);      // O = P V: V is MN-major (dims contiguous)
+        constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(FT_BQ, VD);         // O = P V: V is MN-major (dims contiguous)
         int JU0 = 0, I = 0, J0 = 0;
         FpItem it;
         bool ok = true;
@@ -656,9 +659,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
               if (NBUF == 1 && !mbar_wait(b_sub + SUB_BARS * x + B_SEMPTY + 8 * sb, ((Jg / NBUF) & 1) ^ 1, abort)) return false;
               asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-              for (int k = 0; k < FT_HD / 16; k++)      // 16 dims a step: four steps in each 64-wide block
-                umma_bf16(tmem_base + x * SUB_COLS + sb * 64, umma_desc_sw128(sQ + x * Q_BYTES + (k >> 2) * QA + (k & 3) * 32),
-                          umma_desc_sw128(sK + s * KV_BYTES + (k >> 2) * KA + (k & 3) * 32), idesc_s, k ? 1u : 0u);
+              for (int k = 0; k < KD / 16; k++)         // 16 dims a step: four steps in each 64-wide block
+                if (16 * k < p.hd)
+                  umma_bf16(tmem_base + x * SUB_COLS + sb * 64, umma_desc_sw128(sQ + x * Q_BYTES + (k >> 2) * QA + (k & 3) * 32),
+                            umma_desc_sw128(sK + s * K_BYTES + (k >> 2) * KA + (k & 3) * 32), idesc_s, k ? 1u : 0u);
               umma_commit(b_sub + SUB_BARS * x + 8 * sb);
             }
             if (u == n_union - 1) umma_commit(b_qempty);     // the item's last products that read Q
@@ -676,7 +680,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
               for (int k = 0; k < FT_BK / 16; k++)
                 umma_bf16_ta(tmem_base + x * SUB_COLS + 128, tmem_base + x * SUB_COLS + P_COL0 + a * P_STEP + k * 8,
-                             umma_desc_sw128_mn(sV + s * KV_BYTES + k * 2048, NA > 1 ? KA : 0), idesc_o, (j | k) ? 1u : 0u);
+                             umma_desc_sw128_mn(sV + s * V_BYTES + k * 2048, NV > 1 ? KA : 0), idesc_o, (j | k) ? 1u : 0u);
               umma_commit(b_sub + SUB_BARS * x + B_OFULL + 8 * a);
             }
             if (!ok) break;
@@ -739,7 +743,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
           uint32_t v[32];
 #pragma unroll 1
-          for (int c0 = 0; c0 < FT_HD; c0 += 32) {
+          for (int c0 = 0; c0 < VD; c0 += 32) {
             tmem_ld32(t_lane + 128 + c0, v);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
@@ -779,10 +783,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         const int JUg = JU0 + (t < it.kept ? t : t - it.skip), st = JUg % FT_STAGES, n_valid = max(0, seq_end + 1 - t * FT_BK);
         ok = mbar_wait(b_kvfull + 8 * st, (JUg / FT_STAGES) & 1, abort);
         if (!ok) break;
-        for (int e = q * 32 + lane; e < (FT_BK - n_valid) * 8 * NA; e += 128) {
+        for (int e = q * 32 + lane; e < (FT_BK - n_valid) * 8 * NV; e += 128) {
           int blk = e / ((FT_BK - n_valid) * 8), e1 = e % ((FT_BK - n_valid) * 8);
           int row = n_valid + e1 / 8, c = e1 % 8;
-          *(uint4*)(smem + 2 * Q_BYTES + FT_STAGES * KV_BYTES + st * KV_BYTES + blk * KA + row * 128 + ((c ^ (row & 7)) << 4)) = make_uint4(0, 0, 0, 0);
+          *(uint4*)(smem + 2 * Q_BYTES + FT_STAGES * K_BYTES + st * V_BYTES + blk * KA + row * 128 + ((c ^ (row & 7)) << 4)) = make_uint4(0, 0, 0, 0);
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       }
@@ -799,14 +803,14 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       if (p.sink != nullptr) l = (m_ref == -INFINITY) ? 1.f : l + ft_ex2(p.sink[sb.h] * FT_LOG2E - m_ref * sc);
       float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = p.out + (size_t)(it.row0 + sb.r0 + r) * ((size_t)p.H * FT_HD) + (size_t)sb.h * FT_HD;
+      bf16* dst = p.out + (size_t)(it.row0 + sb.r0 + r) * ((size_t)p.H * p.vd) + (size_t)sb.h * p.vd;
 #pragma unroll 1
-      for (int c0 = 0; c0 < FT_HD; c0 += 32) {
+      for (int c0 = 0; c0 < VD; c0 += 32) {
         uint32_t v[32];
         tmem_ld32(t_lane + 128 + c0, v);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (r < sb.nq) {
-          if (p.gate != nullptr) ft_gate(v, p.gate + (size_t)(it.row0 + sb.r0 + r) * p.gate_ld + (size_t)sb.h * FT_HD + c0);
+          if (p.gate != nullptr) ft_gate(v, p.gate + (size_t)(it.row0 + sb.r0 + r) * p.gate_ld + (size_t)sb.h * p.vd + c0, p.vd - c0);
 #pragma unroll
           for (int c = 0; c < 4; c++) {
             uint4 w;
@@ -815,7 +819,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             __nv_bfloat162 p2 = __floats2bfloat162_rn(__uint_as_float(v[8 * c + 4]) * inv, __uint_as_float(v[8 * c + 5]) * inv);
             __nv_bfloat162 p3 = __floats2bfloat162_rn(__uint_as_float(v[8 * c + 6]) * inv, __uint_as_float(v[8 * c + 7]) * inv);
             w.x = *(uint32_t*)&p0; w.y = *(uint32_t*)&p1; w.z = *(uint32_t*)&p2; w.w = *(uint32_t*)&p3;
-            *(uint4*)(dst + c0 + 8 * c) = w;
+            if (c0 + 8 * c < p.vd) *(uint4*)(dst + c0 + 8 * c) = w;
           }
         }
       }
@@ -851,35 +855,35 @@ static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
   SLLM_RETURN_LAST();
 }
 
-template <int HD, int STAGES>
+template <int KD, int VD, int STAGES>
 static int fp_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FtArgs& a, dim3 grid,
                      cudaStream_t stream) {
   // what the kernel lays out after aligning to 1 KB; one block on an SM
-  constexpr size_t need = 2 * FT_BQ * HD * 2 + 2 * STAGES * FT_BK * HD * 2 + 256;
+  constexpr size_t need = 2 * FT_BQ * KD * 2 + STAGES * FT_BK * (KD + VD) * 2 + 256;
   constexpr size_t room = 232448;
   constexpr size_t smem = need + 1024 <= room ? need + 1024 : room;     // the slack for the alignment, as far as it fits
   static_assert(need <= smem, "the block of this head width does not fit an SM");
   static bool raised = false;
   if (!raised) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_pair_kernel<HD, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_pair_kernel<KD, VD, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     raised = true;
   }
-  attn_prefill_pair_kernel<HD, STAGES><<<grid, FP_THREADS, smem, stream>>>(mq, mk, mv, a, (uint32_t)smem);
+  attn_prefill_pair_kernel<KD, VD, STAGES><<<grid, FP_THREADS, smem, stream>>>(mq, mk, mv, a, (uint32_t)smem);
   SLLM_RETURN_LAST();
 }
 
-// q: [T, q_ld] rotated queries (head h at columns h*hd); out: [T, H*hd]; kpages/vpages:
-// [n_pages][G][64][hd] with n_pages the number of pages the storage holds; hd 64 or 128.
+// q: [T, q_ld] rotated queries (head h at columns h*hd); out: [T, H*vd]; kpages [n_pages][G][64][hd], vpages
+// [n_pages][G][64][vd] with n_pages the number of pages the storage holds; hd and vd multiples of 8 up to 128.
 SLLM_EXPORT int sllm_attn_prefill_tc_bf16(const void* q, int q_ld, int T, void* out, const int* seq_start, const int* seq_pos0,
                                           const int* block_table, int max_pages, const void* kpages, const void* vpages,
-                                          long long n_pages, int B, int max_new, int H, int G, int hd, int window, int keep, float scale,
+                                          long long n_pages, int B, int max_new, int H, int G, int hd, int vd, int window, int keep, float scale,
                                           float softcap, const float* sink, const void* gate, int gate_ld, int* err,
                                           cudaStream_t stream) {
   if (B <= 0 || max_new <= 0) return 0;
-  if ((hd != 64 && hd != 128) || G < 1 || H % G != 0 || (q_ld & 7) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
+  if (hd < 8 || hd > 128 || hd % 8 || vd < 8 || vd > 128 || vd % 8 || q_ld < H * hd || G < 1 || H % G != 0 || (q_ld & 7) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
       ((uintptr_t)kpages & 15) || ((uintptr_t)vpages & 15) || keep < 0 ||
-      (gate && (((uintptr_t)gate & 15) || (gate_ld & 7) || gate_ld < H * hd)))
+      (gate && (((uintptr_t)gate & 15) || (gate_ld & 7) || gate_ld < H * vd)))
     return SLLM_ERR_ARG;
   long long kv_rows = n_pages * G * FT_BK;
   if (kv_rows <= 0 || kv_rows > 0x7fffffffLL) return SLLM_ERR_ARG;
@@ -888,7 +892,7 @@ SLLM_EXPORT int sllm_attn_prefill_tc_bf16(const void* q, int q_ld, int T, void* 
   if (rc) return rc;
   rc = tc_make_map(&mk, kpages, (int)kv_rows, hd, hd, FT_BK);
   if (rc) return rc;
-  rc = tc_make_map(&mv, vpages, (int)kv_rows, hd, hd, FT_BK);
+  rc = tc_make_map(&mv, vpages, (int)kv_rows, vd, vd, FT_BK);
   if (rc) return rc;
   int n_qt = (max_new + FT_BQ - 1) / FT_BQ;
   long long n_items = (long long)H * n_qt * B;
@@ -900,16 +904,18 @@ SLLM_EXPORT int sllm_attn_prefill_tc_bf16(const void* q, int q_ld, int T, void* 
     if (e == cudaSuccess) e = cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev);
     if (e != cudaSuccess) return (int)e;
   }
-  if (hd == 64) {
-    FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, window, keep, scale, err, n_qt, B, (int)n_items, 0, softcap, sink,
+  if (hd <= 64 && vd <= 64) {
+    FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, hd, vd, window, keep, scale, err, n_qt, B, (int)n_items, 0, softcap, sink,
              (const bf16*)gate, gate_ld};
     dim3 grid((unsigned)(n_items < 2LL * sm_count ? n_items : 2LL * sm_count));     // two blocks per SM that stay
     return ft_launch<64, 3>(mq, mk, mv, a, grid, stream);
   }
   int pair_heads = ((H / G) % 2 == 0) ? 1 : 0;
   n_items = pair_heads ? (long long)(H / 2) * n_qt * B : (long long)H * ((n_qt + 1) / 2) * B;
-  FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, window, keep, scale, err, n_qt, B, (int)n_items, pair_heads, softcap, sink,
+  FtArgs a{(bf16*)out, seq_start, seq_pos0, block_table, max_pages, H, G, hd, vd, window, keep, scale, err, n_qt, B, (int)n_items, pair_heads, softcap, sink,
            (const bf16*)gate, gate_ld};
   dim3 grid((unsigned)(n_items < (long long)sm_count ? n_items : (long long)sm_count));       // one block per SM that stays
-  return fp_launch<128, 4>(mq, mk, mv, a, grid, stream);
+  if (vd <= 64) return fp_launch<128, 64, 5>(mq, mk, mv, a, grid, stream);
+  if (hd <= 64) return fp_launch<64, 128, 5>(mq, mk, mv, a, grid, stream);
+  return fp_launch<128, 128, 4>(mq, mk, mv, a, grid, stream);
 }

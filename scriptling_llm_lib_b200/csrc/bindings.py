@@ -468,25 +468,31 @@ class TensorCoreGemm:
 
 
 class PrefillAttentionTC:
-    """tcgen05 causal attention of a prompt step over the paged cache (bfloat16, head width 64 or 128)."""
+    """tcgen05 causal attention of a prompt step over the paged cache (bfloat16; keys and values of one width, 64 or 128, at
+    full speed, or any two multiples of 8 up to 128, filled up with zeros on the chip)."""
     HEAD_DIMS = (64, 128)
+
+    @staticmethod
+    def takes(key_dim: int, value_dim: int) -> bool:
+        return all(w % 8 == 0 and 8 <= w <= 128 for w in (key_dim, value_dim))
 
     def __init__(self):
         self.lib = load_library("attn_prefill_tcgen05")
         self.lib.sllm_attn_prefill_tc_bf16.restype = c_int
 
     def attn(self, q, out, seq_start, seq_pos0, block_table, kpages, vpages, n_seqs, max_new, n_heads, n_kv, head_dim,
-             window, scale, err_flag, softcap=None, sink=None, keep=0, gate=None):
-        """`softcap`: a score s becomes softcap * tanh(s / softcap) before the softmax; `sink` float32 [n_heads]: exp(sink[h])
+             window, scale, err_flag, softcap=None, sink=None, keep=0, gate=None, v_dim=None):
+        """`v_dim`: the values' width where it is not the keys'. `softcap`: a score s becomes softcap * tanh(s / softcap) before the softmax; `sink` float32 [n_heads]: exp(sink[h])
         joins head h's denominator with no key and no value; `keep`: the first positions of a sequence that stay visible behind
-        the window; `gate`: bfloat16 [T, n_heads * head_dim] (a column slice), whose sigmoid multiplies the output."""
-        gp, gl = _gate_args(gate, q.shape[0], n_heads * head_dim)
+        the window; `gate`: bfloat16 [T, n_heads * v_dim] (a column slice), whose sigmoid multiplies the output."""
+        v_dim = v_dim or head_dim
+        gp, gl = _gate_args(gate, q.shape[0], n_heads * v_dim)
         _check(self.lib.sllm_attn_prefill_tc_bf16(
             _ptr(q, torch.bfloat16, "q"), c_int(q.shape[1]), c_int(q.shape[0]), _ptr(out, torch.bfloat16, "out"),
             _ptr(seq_start, torch.int32, "seq_start"), _ptr(seq_pos0, torch.int32, "seq_pos0"),
             _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]),
             _ptr(kpages, torch.bfloat16, "kpages"), _ptr(vpages, torch.bfloat16, "vpages"), c_longlong(kpages.shape[0]),
-            c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(window or 0), c_int(keep),
+            c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_int(v_dim), c_int(window or 0), c_int(keep),
             c_float(scale), c_float(softcap or 0.0), _ptr(sink, torch.float32, "sink"), gp, gl, _ptr(err_flag, torch.int32, "err_flag"),
             _stream()), "attn_prefill_tc")
 
@@ -551,7 +557,7 @@ class DecodeKernels:
         self.lib = load_library("decode_bf16")
         for n in ("sllm_gemm_small_m_bf16", "sllm_gemm_small_m_fold_bf16", "sllm_attn_decode_bf16",
                   "sllm_attn_decode_merged_bf16", "sllm_attn_decode_rope_bf16", "sllm_attn_decode_capped_bf16",
-                  "sllm_attn_decode_general_bf16"):
+                  "sllm_attn_decode_general_bf16", "sllm_gemm_small_m_act_bf16"):
             getattr(self.lib, n).restype = c_int
         self.lib.sllm_attn_decode_scratch_bytes.restype = c_longlong
         self.lib.sllm_attn_decode_uses_mma.restype = c_int
@@ -623,6 +629,16 @@ class DecodeKernels:
             _ptr(w, torch.bfloat16, "w"), _ptr(out, None, "out"), c_int(M), c_int(N), c_int(K), c_int(a.stride(0)),
             c_int(w.stride(0)), c_int(out.stride(-2)), c_int(1 if out.dtype == torch.float32 else 0),
             c_int(1 if swiglu else 0), c_int(ksplit), _stream()), "gemm_small_m")
+
+    def gemm_small_m_act(self, a, w, out, act: str):
+        """out[M, N] (bfloat16) = act(a @ w^T), the activation on the float sums (names as `TensorCoreGemm.ACTS`)."""
+        M, K = a.shape
+        N = w.shape[0]
+        if w.shape[1] != K or tuple(out.shape) != (M, N) or out.dtype != torch.bfloat16 or a.dtype != torch.bfloat16 or a.stride(1) != 1:
+            raise KernelError(f"gemm_small_m_act shapes: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} {out.dtype}")
+        _check(self.lib.sllm_gemm_small_m_act_bf16(
+            c_void_p(a.data_ptr()), _ptr(w, torch.bfloat16, "w"), _ptr(out, torch.bfloat16, "out"), c_int(M), c_int(N), c_int(K),
+            c_int(a.stride(0)), c_int(w.stride(0)), c_int(N), c_int(TensorCoreGemm.ACTS[act]), _stream()), "gemm_small_m_act")
 
     def _gemm_small_m_fold(self, a, w, out, swiglu, owed, fold):
         M, K = a.shape

@@ -56,6 +56,13 @@ template <> __device__ __forceinline__ float from_f32<float>(float v) { return v
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
 __device__ __forceinline__ float sigmoid_of(float v) { return 1.0f / (1.0f + expf(-v)); }
+// the feed-forwards' activations: 0 none, 1 the tanh form of gelu, 2 the square of relu, 3 silu
+__device__ __forceinline__ float act_of(int kind, float z) {
+  if (kind == 0) return z;
+  if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (kind == 2) return z > 0.f ? z * z : 0.f;
+  return z * sigmoid_of(z);
+}
 
 // weights of a norm may be stored in bfloat16 or float32 whatever the activation type
 __device__ __forceinline__ float load_w(const void* w, int is_f32, int j) {

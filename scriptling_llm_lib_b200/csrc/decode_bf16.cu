@@ -66,6 +66,7 @@ struct SmFold {
   const float* norm_w;
   bf16* xb;
   float* sumsq_out;
+  int act;              // of the plain epilogue with bfloat16 output (common.cuh: act_of)
 };
 
 __device__ __forceinline__ float ld_dep_f32(const float* p) {      // of data an earlier kernel of the stream wrote
@@ -203,7 +204,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, void
     if (EPI == SM_EPI_STORE) {
       if (feat < N && tok < M) {
         if (out_f32) ((float*)y)[((size_t)blockIdx.y * M + tok) * ldy + feat] = s;
-        else ((bf16*)y)[(size_t)tok * ldy + feat] = __float2bfloat16_rn(s);
+        else ((bf16*)y)[(size_t)tok * ldy + feat] = __float2bfloat16_rn(act_of(f.act, s));
       }
     } else if (EPI == SM_EPI_RESID) {
       float sq = 0.f;
@@ -309,10 +310,9 @@ static int small_m_launch(const bf16* x, const bf16* W, void* y, int M, int N, i
 // epilogue 2 (M <= 16): y is the float residual stream [M][ldy], which receives the product; xb[M][N] and
 // sumsq_out[ceil(N/16)][M] receive what the product after the following norm needs (see SmFold).
 // sumsq_in (or null), n_in, width_in, eps_in: the scale owed to the rows of x (see SmFold).
-SLLM_EXPORT int sllm_gemm_small_m_fold_bf16(const void* x, const void* W, void* y, int M, int N, int K, int ldx, int ldw,
-                                            int ldy, int out_f32, int epilogue, int ksplit, const float* sumsq_in, int n_in,
-                                            int width_in, float eps_in, const float* norm_w, void* xb, float* sumsq_out,
-                                            cudaStream_t stream) {
+static int gemm_small_m_dispatch(const void* x, const void* W, void* y, int M, int N, int K, int ldx, int ldw, int ldy, int out_f32,
+                                 int epilogue, int ksplit, const float* sumsq_in, int n_in, int width_in, float eps_in,
+                                 const float* norm_w, void* xb, float* sumsq_out, int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || ((uintptr_t)x & 15) || ((uintptr_t)W & 15)) return SLLM_ERR_ARG;
   if (epilogue == SM_EPI_SWIGLU && ((N & 15) || out_f32 || ksplit != 1)) return SLLM_ERR_ARG;
@@ -322,7 +322,7 @@ SLLM_EXPORT int sllm_gemm_small_m_fold_bf16(const void* x, const void* W, void* 
   if (sumsq_in && (n_in < 1 || width_in < 1)) return SLLM_ERR_ARG;
   const bf16* xp = (const bf16*)x;
   const bf16* wp = (const bf16*)W;
-  SmFold f{sumsq_in, n_in, sumsq_in ? 1.0f / (float)width_in : 0.f, eps_in, (float*)y, norm_w, (bf16*)xb, sumsq_out};
+  SmFold f{sumsq_in, n_in, sumsq_in ? 1.0f / (float)width_in : 0.f, eps_in, (float*)y, norm_w, (bf16*)xb, sumsq_out, act};
 #define SM_CASE(NT)                                                                                                          \
   return epilogue == SM_EPI_SWIGLU  ? small_m_launch<NT, SM_EPI_SWIGLU>(xp, wp, y, M, N, K, ldx, ldw, ldy, 0, 1, f, stream)  \
          : epilogue == SM_EPI_RESID ? small_m_launch<(NT <= 2 ? NT : 2), SM_EPI_RESID>(xp, wp, y, M, N, K, ldx, ldw, ldy, 1, 1, f, stream) \
@@ -332,6 +332,21 @@ SLLM_EXPORT int sllm_gemm_small_m_fold_bf16(const void* x, const void* W, void* 
   if (M <= 32) { SM_CASE(4); }
   SM_CASE(8);
 #undef SM_CASE
+}
+
+SLLM_EXPORT int sllm_gemm_small_m_fold_bf16(const void* x, const void* W, void* y, int M, int N, int K, int ldx, int ldw,
+                                            int ldy, int out_f32, int epilogue, int ksplit, const float* sumsq_in, int n_in,
+                                            int width_in, float eps_in, const float* norm_w, void* xb, float* sumsq_out,
+                                            cudaStream_t stream) {
+  return gemm_small_m_dispatch(x, W, y, M, N, K, ldx, ldw, ldy, out_f32, epilogue, ksplit, sumsq_in, n_in, width_in, eps_in, norm_w,
+                               xb, sumsq_out, 0, stream);
+}
+
+// y[M,N] = act(x W^T) in bfloat16, the activation (common.cuh: act_of) on the float sums
+SLLM_EXPORT int sllm_gemm_small_m_act_bf16(const void* x, const void* W, void* y, int M, int N, int K, int ldx, int ldw, int ldy, int act,
+                                           cudaStream_t stream) {
+  if (act < 0 || act > 3) return SLLM_ERR_ARG;
+  return gemm_small_m_dispatch(x, W, y, M, N, K, ldx, ldw, ldy, 0, SM_EPI_STORE, 1, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, act, stream);
 }
 
 SLLM_EXPORT int sllm_gemm_small_m_bf16(const void* x, const void* W, void* y, int M, int N, int K, int ldx, int ldw,

@@ -64,33 +64,79 @@ template <typename A, int V> __device__ __forceinline__ void st_pack(A* p, const
 }
 
 #define QKS_WARPS 8
-// V elements a lane and access (4 where widths and addresses allow, else 1). A warp takes a head at a time; a head's
-// elements stay in registers between the sum of squares and the stores (heads of up to 512).
-template <typename A, int V>
+// V elements a lane and access (4 where widths and addresses allow, else 1), NIT accesses to a head. A warp takes NB heads at
+// a time, whose loads are all asked for before the first is used and whose elements stay in registers up to the stores; with
+// a norm over the whole projection they stay over the block's two sums as well where one such batch a warp covers all heads.
+template <typename A, int V, int NIT, int NB>
 __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreArgs p) {
-  constexpr int NIT = 16 / V;
   __shared__ float red[2][QKS_WARPS];
   extern __shared__ float qks_row[];             // with a rotation: hd floats a warp
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int hd = p.hd, vd = p.vd, QW = p.H * hd, KW = p.G * hd;
+  const int H = p.H, heads = p.H + p.G, hd = p.hd, vd = p.vd, QW = H * hd, KW = p.G * hd, VW = p.G * vd;
   const int pos = p.tok_pos[t];
   const size_t row = (size_t)t * p.ld;
-  float rq = 1.f, rk = 1.f;
-  if (!p.per_head && (p.qw || p.kw)) {
-    float sq = 0.f, sk = 0.f;
-    for (int j = threadIdx.x * V; j < QW + KW; j += QKS_WARPS * 32 * V) {
-      Pack<V> x = ld_pack_flag<A, V>(p.c, p.c_f32, row + j);
-      if (p.bias) {
-        Pack<V> b = ld_pack<V>(p.bias + j);
+  size_t page_slot = 0;
+  if (p.G > 0) {
+    int page = p.block_table[(size_t)p.tok_seq[t] * p.max_pages + pos / SLLM_PAGE];
+    page_slot = (size_t)page * p.G * SLLM_PAGE + (pos % SLLM_PAGE);     // + g * PAGE, times the head width
+  }
+  // the block's first values are on their way while queries and keys are worked
+  const int e0 = threadIdx.x * V;
+  Pack<V> val;
+  if (e0 < VW) val = ld_pack_flag<A, V>(p.c, p.c_f32, row + QW + KW + e0);
+
+  Pack<V> x[NB][NIT];
+  auto load = [&](int first) {                   // heads first, first + QKS_WARPS, ...
 #pragma unroll
-        for (int i = 0; i < V; i++) x.f[i] += b.f[i];
+    for (int n = 0; n < NB; n++) {
+      const int head = first + n * QKS_WARPS;
+#pragma unroll
+      for (int it = 0; it < NIT; it++) {
+        const int j = (it * 32 + lane) * V;
+        if (head < heads && j < hd) x[n][it] = ld_pack_flag<A, V>(p.c, p.c_f32, row + head * hd + j);
       }
-      float s = 0.f;
+    }
+    if (p.bias) {
 #pragma unroll
-      for (int i = 0; i < V; i++) s = fmaf(x.f[i], x.f[i], s);
-      if (j < QW) sq += s; else sk += s;
+      for (int n = 0; n < NB; n++) {
+        const int head = first + n * QKS_WARPS;
+#pragma unroll
+        for (int it = 0; it < NIT; it++) {
+          const int j = (it * 32 + lane) * V;
+          if (head < heads && j < hd) {
+            const Pack<V> b = ld_pack<V>(p.bias + head * hd + j);
+#pragma unroll
+            for (int i = 0; i < V; i++) x[n][it].f[i] += b.f[i];
+          }
+        }
+      }
+    }
+  };
+  auto squares = [&](int n, int head) -> float {  // this lane's share of a head's sum
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < NIT; it++)
+      if (head < heads && (it * 32 + lane) * V < hd) {
+#pragma unroll
+        for (int i = 0; i < V; i++) ss = fmaf(x[n][it].f[i], x[n][it].f[i], ss);
+      }
+    return ss;
+  };
+  constexpr int BATCH = QKS_WARPS * NB;
+  const bool whole = !p.per_head && (p.qw || p.kw);
+  float rq = 1.f, rk = 1.f;
+  if (whole) {
+    float sq = 0.f, sk = 0.f;
+    for (int first = warp; first < heads; first += BATCH) {
+      load(first);
+#pragma unroll
+      for (int n = 0; n < NB; n++) {
+        const int head = first + n * QKS_WARPS;
+        const float ss = squares(n, head);
+        if (head < H) sq += ss; else sk += ss;
+      }
     }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
@@ -102,83 +148,69 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreAr
     if (p.qw) rq = 1.0f / sqrtf(sq / (float)QW + p.eps);
     if (p.kw && KW > 0) rk = 1.0f / sqrtf(sk / (float)KW + p.eps);
   }
-  size_t page_slot = 0;
-  if (p.G > 0) {
-    int page = p.block_table[(size_t)p.tok_seq[t] * p.max_pages + pos / SLLM_PAGE];
-    page_slot = (size_t)page * p.G * SLLM_PAGE + (pos % SLLM_PAGE);     // + g * PAGE, times the head width
-  }
   const int half = p.rot >> 1;
   const float2* csr = p.cs + (size_t)pos * half;
   float* wrow = qks_row + warp * hd;
-  for (int head = warp; head < p.H + p.G; head += QKS_WARPS) {
-    const bool is_q = head < p.H;
-    const int col = head * hd;                                         // the key part follows the query part directly
-    const void* w = is_q ? p.qw : p.kw;
-    const int wc = p.per_head ? 0 : is_q ? col : col - QW;
-    Pack<V> x[NIT];
-    float ss = 0.f;
+  for (int first = warp; first < heads; first += BATCH) {
+    if (!(whole && heads <= BATCH)) load(first);
 #pragma unroll
-    for (int it = 0; it < NIT; it++) {
-      const int j = (it * 32 + lane) * V;
-      if (j >= hd) break;
-      x[it] = ld_pack_flag<A, V>(p.c, p.c_f32, row + col + j);
-      if (p.bias) {
-        Pack<V> b = ld_pack<V>(p.bias + col + j);
+    for (int n = 0; n < NB; n++) {
+      const int head = first + n * QKS_WARPS;
+      if (head >= heads) break;
+      const bool is_q = head < H;
+      const int col = head * hd;                                         // the key part follows the query part directly
+      const void* w = is_q ? p.qw : p.kw;
+      const int wc = p.per_head ? 0 : is_q ? col : col - QW;
+      float r = is_q ? rq : rk;
+      if (p.per_head && w) r = 1.0f / sqrtf(warp_sum(squares(n, head)) / (float)hd + p.eps);
+      A* dst = is_q ? (A*)p.q_out + (size_t)t * p.ldq + col : (A*)p.kpages + (page_slot + (size_t)(head - H) * SLLM_PAGE) * hd;
 #pragma unroll
-        for (int i = 0; i < V; i++) x[it].f[i] += b.f[i];
+      for (int it = 0; it < NIT; it++) {
+        const int j = (it * 32 + lane) * V;
+        if (j >= hd) break;
+        if (w) {
+          const Pack<V> ww = ld_pack_flag<bf16, V>(w, p.w_f32, wc + j);
+#pragma unroll
+          for (int i = 0; i < V; i++) x[n][it].f[i] = x[n][it].f[i] * r * ww.f[i];
+        }
+        if (p.rot > 0) {
+#pragma unroll
+          for (int i = 0; i < V; i++) wrow[j + i] = x[n][it].f[i];
+        } else {
+          st_pack<A, V>(dst + j, x[n][it]);
+        }
       }
-#pragma unroll
-      for (int i = 0; i < V; i++) ss = fmaf(x[it].f[i], x[it].f[i], ss);
-    }
-    float r = is_q ? rq : rk;
-    if (p.per_head && w) r = 1.0f / sqrtf(warp_sum(ss) / (float)hd + p.eps);
-    A* dst = is_q ? (A*)p.q_out + (size_t)t * p.ldq + col : (A*)p.kpages + (page_slot + (size_t)(head - p.H) * SLLM_PAGE) * hd;
-#pragma unroll
-    for (int it = 0; it < NIT; it++) {
-      const int j = (it * 32 + lane) * V;
-      if (j >= hd) break;
-      if (w) {
-        Pack<V> ww = ld_pack_flag<bf16, V>(w, p.w_f32, wc + j);
-#pragma unroll
-        for (int i = 0; i < V; i++) x[it].f[i] = x[it].f[i] * r * ww.f[i];
+      if (p.rot > 0) {                                                   // a lane turns a pair; the rest passes as it is
+        __syncwarp();
+        for (int i = lane; i < half; i += 32) {
+          const int i0 = p.interleaved ? 2 * i : i, i1 = p.interleaved ? 2 * i + 1 : i + half;
+          const float2 a = csr[i];
+          const float x0 = wrow[i0], x1 = wrow[i1];
+          dst[i0] = from_f32<A>(x0 * a.x - x1 * a.y);
+          dst[i1] = from_f32<A>(x1 * a.x + x0 * a.y);
+        }
+        for (int j = p.rot + lane; j < hd; j += 32) dst[j] = from_f32<A>(wrow[j]);
+        __syncwarp();
       }
-      if (p.rot > 0) {
-#pragma unroll
-        for (int i = 0; i < V; i++) wrow[j + i] = x[it].f[i];
-      } else {
-        st_pack<A, V>(dst + j, x[it]);
-      }
-    }
-    if (p.rot > 0) {                                                   // a lane turns a pair; the rest passes as it is
-      __syncwarp();
-      for (int i = lane; i < half; i += 32) {
-        const int i0 = p.interleaved ? 2 * i : i, i1 = p.interleaved ? 2 * i + 1 : i + half;
-        const float2 a = csr[i];
-        const float x0 = wrow[i0], x1 = wrow[i1];
-        dst[i0] = from_f32<A>(x0 * a.x - x1 * a.y);
-        dst[i1] = from_f32<A>(x1 * a.x + x0 * a.y);
-      }
-      for (int j = p.rot + lane; j < hd; j += 32) dst[j] = from_f32<A>(wrow[j]);
-      __syncwarp();
     }
   }
-  // values, one pass of the block over all heads
-  A* vm = (A*)p.vmix + (size_t)t * p.G * vd;
-  for (int e = threadIdx.x * V; e < p.G * vd; e += QKS_WARPS * 32 * V) {
+  // values, the block over all heads
+  A* vm = (A*)p.vmix + (size_t)t * VW;
+  for (int e = e0; e < VW; e += QKS_WARPS * 32 * V) {
     const int g = e / vd, j = e % vd;
-    Pack<V> x = ld_pack_flag<A, V>(p.c, p.c_f32, row + QW + KW + e);
+    if (e != e0) val = ld_pack_flag<A, V>(p.c, p.c_f32, row + QW + KW + e);
     if (p.bias) {
-      Pack<V> b = ld_pack<V>(p.bias + QW + KW + e);
+      const Pack<V> b = ld_pack<V>(p.bias + QW + KW + e);
 #pragma unroll
-      for (int i = 0; i < V; i++) x.f[i] += b.f[i];
+      for (int i = 0; i < V; i++) val.f[i] += b.f[i];
     }
-    if (p.mix_mode == 1) st_pack<A, V>(vm + e, x);
+    if (p.mix_mode == 1) st_pack<A, V>(vm + e, val);
     if (p.mix_mode == 2) {
-      Pack<V> f = ld_pack<V>((const A*)vm + e);
+      const Pack<V> f = ld_pack<V>((const A*)vm + e);
 #pragma unroll
-      for (int i = 0; i < V; i++) x.f[i] = (1.0f - p.lam) * x.f[i] + p.lam * f.f[i];
+      for (int i = 0; i < V; i++) val.f[i] = (1.0f - p.lam) * val.f[i] + p.lam * f.f[i];
     }
-    st_pack<A, V>((A*)p.vpages + (page_slot + (size_t)g * SLLM_PAGE) * vd + j, x);
+    st_pack<A, V>((A*)p.vpages + (page_slot + (size_t)g * SLLM_PAGE) * vd + j, val);
   }
 }
 
@@ -564,64 +596,91 @@ __global__ void add_rms_normed_kernel(float* x, const void* y, int y_f32, int P,
     out[(size_t)blockIdx.x * d + j] = from_f32<A>(rowbuf[j] * r2 * load_w(w2, w2_f32, j));
 }
 
-// four columns a thread (d a multiple of four); the partial sums are added in the same order
-template <typename A>
-__global__ void add_rms_normed_vec_kernel(float* x, const void* y, int y_f32, int P, int T, const float* yb,
-                                          const void* __restrict__ w, int w_f32, int d, float eps, const int* __restrict__ rows,
-                                          const void* __restrict__ w2, int w2_f32, float eps2, A* out,
-                                          const float* __restrict__ vec, const float* __restrict__ b2, float alpha2) {
-  extern __shared__ __align__(16) float rowbuf[];
-  __shared__ float red[32];
+// The same for rows that fit a block's registers, NV accesses of four columns a thread: the stream's row is asked for together
+// with the addend, and neither passes through shared memory.
+struct RmsAddArgs {
+  float* x; const void* y; int y_f32, P, T; const float* yb; const void* w; int w_f32, d; float eps; const int* rows;
+  const void* w2; int w2_f32; float eps2; void* out; const float* vec; const float* b2; float alpha2;
+};
+__device__ __forceinline__ float4 load_w4(const void* w, int is_f32, int j) {
+  return is_f32 ? *(const float4*)((const float*)w + j) : ld4((const bf16*)w + j);
+}
+__device__ __forceinline__ float dot4(const float4& a) { return fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, a.w * a.w))); }
+
+template <typename A, int NV>
+__global__ void __launch_bounds__(NV == 4 ? 512 : 1024) add_rms_normed_reg_kernel(RmsAddArgs p) {
+  __shared__ float red[2][32];
   pdl_launch_dependents();
+  const int d = p.d, step = blockDim.x * 4, j0 = threadIdx.x * 4;
+  float4 w[NV];
+#pragma unroll
+  for (int n = 0; n < NV; n++)
+    if (j0 + n * step < d) w[n] = load_w4(p.w, p.w_f32, j0 + n * step);      // a weight: no kernel of the step writes it
   pdl_wait();
-  int t = rows ? rows[blockIdx.x] : blockIdx.x;
-  float ss = 0.f;
-  for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int p = 0; p < P; p++) {
-      float4 a = ld4f<A>(y, y_f32, ((size_t)p * T + t) * d + j);
-      v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+  const int t = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+  float* xr = p.x + (size_t)t * d;
+  float4 x[NV], y[NV];
+#pragma unroll
+  for (int n = 0; n < NV; n++) {
+    const int j = j0 + n * step;
+    if (j < d) {
+      y[n] = ld4f<A>(p.y, p.y_f32, (size_t)t * d + j);
+      x[n] = *(const float4*)(xr + j);
     }
-    if (yb) {
-      float4 b = *(const float4*)(yb + j);
+  }
+  for (int q = 1; q < p.P; q++) {
+#pragma unroll
+    for (int n = 0; n < NV; n++) {
+      const int j = j0 + n * step;
+      if (j < d) {
+        const float4 a = ld4f<A>(p.y, p.y_f32, ((size_t)q * p.T + t) * d + j);
+        y[n].x += a.x; y[n].y += a.y; y[n].z += a.z; y[n].w += a.w;
+      }
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; n++) {
+    const int j = j0 + n * step;
+    if (j >= d) continue;
+    if (p.yb) {
+      const float4 b = *(const float4*)(p.yb + j);
+      y[n].x += b.x; y[n].y += b.y; y[n].z += b.z; y[n].w += b.w;
+    }
+    ss += dot4(y[n]);
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, red[0]) / (float)d + p.eps);
+  A* out = (A*)p.out + (size_t)blockIdx.x * d;
+  float ss2 = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; n++) {
+    const int j = j0 + n * step;
+    if (j >= d) continue;
+    float4 v = x[n];
+    v.x += y[n].x * r * w[n].x; v.y += y[n].y * r * w[n].y; v.z += y[n].z * r * w[n].z; v.w += y[n].w * r * w[n].w;
+    if (p.vec) {
+      const float4 b = *(const float4*)(p.vec + j);
       v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
     }
-    *(float4*)(rowbuf + j) = v;
-    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    *(float4*)(xr + j) = v;
+    x[n] = v;
+    if (p.out && !p.w2) st4(out + j, v);
+    ss2 += dot4(v);
   }
-  float r = 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps);
-  float ss2 = 0.f;
-  for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
-    float4 v = *(const float4*)(rowbuf + j);
-    float4 xv = *(const float4*)(x + (size_t)t * d + j);
-    xv.x += v.x * r * load_w(w, w_f32, j);
-    xv.y += v.y * r * load_w(w, w_f32, j + 1);
-    xv.z += v.z * r * load_w(w, w_f32, j + 2);
-    xv.w += v.w * r * load_w(w, w_f32, j + 3);
-    if (vec) {
-      float4 b = *(const float4*)(vec + j);
-      xv.x += b.x; xv.y += b.y; xv.z += b.z; xv.w += b.w;
+  if (!p.out || !p.w2) return;
+  const float r2 = p.b2 ? 0.f : 1.0f / sqrtf(block_sum(ss2, red[1]) / (float)d + p.eps2);
+#pragma unroll
+  for (int n = 0; n < NV; n++) {
+    const int j = j0 + n * step;
+    if (j >= d) continue;
+    const float4 v = x[n], u = load_w4(p.w2, p.w2_f32, j);
+    if (p.b2) {
+      const float4 b = *(const float4*)(p.b2 + j);
+      st4(out + j, make_float4(tanhf(p.alpha2 * v.x) * u.x + b.x, tanhf(p.alpha2 * v.y) * u.y + b.y, tanhf(p.alpha2 * v.z) * u.z + b.z,
+                               tanhf(p.alpha2 * v.w) * u.w + b.w));
+    } else {
+      st4(out + j, make_float4(v.x * r2 * u.x, v.y * r2 * u.y, v.z * r2 * u.z, v.w * r2 * u.w));
     }
-    *(float4*)(x + (size_t)t * d + j) = xv;
-    if (out && !w2) { st4(out + (size_t)blockIdx.x * d + j, xv); continue; }
-    *(float4*)(rowbuf + j) = xv;
-    ss2 += xv.x * xv.x + xv.y * xv.y + xv.z * xv.z + xv.w * xv.w;
-  }
-  if (!out || !w2) return;
-  if (b2) {
-    for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
-      float4 v = *(const float4*)(rowbuf + j);
-      float4 ww = *(const float4*)((const float*)w2 + j), bb = *(const float4*)(b2 + j);
-      st4(out + (size_t)blockIdx.x * d + j, make_float4(tanhf(alpha2 * v.x) * ww.x + bb.x, tanhf(alpha2 * v.y) * ww.y + bb.y,
-                                                        tanhf(alpha2 * v.z) * ww.z + bb.z, tanhf(alpha2 * v.w) * ww.w + bb.w));
-    }
-    return;
-  }
-  float r2 = 1.0f / sqrtf(block_sum(ss2, red) / (float)d + eps2);
-  for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
-    float4 v = *(const float4*)(rowbuf + j);
-    st4(out + (size_t)blockIdx.x * d + j, make_float4(v.x * r2 * load_w(w2, w2_f32, j), v.y * r2 * load_w(w2, w2_f32, j + 1),
-                                                      v.z * r2 * load_w(w2, w2_f32, j + 2), v.w * r2 * load_w(w2, w2_f32, j + 3)));
   }
 }
 

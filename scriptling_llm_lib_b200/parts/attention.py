@@ -45,8 +45,8 @@ same sink logit for every head as a constant instead of a stored one (0: one is 
 layers that share a `group` mix their values with those the group's first layer projected for the same token, v <- (1 - lam)
 v + lam v_first with lam a stored number, before they are cached; the first layer's values stay at hand for the step.
 With any of these, attention runs on the kernels that know keys and values of different widths, the window with kept
-positions and the sink: in bfloat16 the tcgen05 prompt kernels (heads of 64 and 128), the mma.sync prompt and decode
-kernels (keys up to 256, values up to 128, multiples of 8), else and in 32-bit the generic ones.
+positions and the sink: in bfloat16 the tcgen05 prompt kernels (widths up to 128 in multiples of 8), the mma.sync prompt and
+decode kernels (keys up to 256, values up to 128, multiples of 8), else and in 32-bit the generic ones.
 
 The position encoding is optional (`position=None`: queries and keys as projected). Storing keys
 and values in the cache is this mixer's own step, whatever the encoding: for an encoding that is a
@@ -305,9 +305,9 @@ class Attention(Mixer):
             scratch = torch.empty((ctx.n_seqs * H * n_split * (vd + 2),), dtype=torch.float32, device=q.device)
             k.decode.attn_decode_general(q, attn, ctx.seq_pos0, block_table, kpages, vpages, scratch, ctx.engine.tickets(ctx.n_seqs * G),
                                          ctx.n_seqs, H, G, hd, vd, self.span, self.scale, n_split, gate=fused_gate, **options)
-        elif not ctx.is_decode and bf16 and hd == vd and hd in PrefillAttentionTC.HEAD_DIMS:
+        elif not ctx.is_decode and bf16 and PrefillAttentionTC.takes(hd, vd):
             k.prefill_attention_tc.attn(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, H, G,
-                                        hd, self.span, self.scale, ctx.err_flag, gate=fused_gate, **options)
+                                        hd, self.span, self.scale, ctx.err_flag, gate=fused_gate, v_dim=vd, **options)
         elif not ctx.is_decode and bf16 and PrefillAttentionMMA.takes(hd, vd):
             k.prefill_attention_mma.attn(q, hd, attn, vd, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs,
                                          ctx.max_new, H, G, hd, vd, self.span, self.scale, gate=fused_gate, **options)

@@ -75,6 +75,10 @@ class ActFeedForward(FeedForward):
                 h = torch.empty((x.shape[0], self.intermediate), dtype=x.dtype, device=x.device)
                 tc.gemm_act(x, w, h, ctx.err_flag, self.act)
                 return self.down.forward(h, ctx, partials_ok=True)
+            if not tc.prefers_skinny(x, w, "plain", ctx.engine.sm_count) and ctx.kernels.decode.prefers(x, w, ctx.engine.sm_count):
+                h = torch.empty((x.shape[0], self.intermediate), dtype=x.dtype, device=x.device)
+                ctx.kernels.decode.gemm_small_m_act(x, w, h, self.act)
+                return self.down.forward(h, ctx, partials_ok=True)
         h = self.up.forward(x, ctx)
         ctx.kernels.mix.act_inplace(h, self.act)
         return self.down.forward(h, ctx, partials_ok=True)
