@@ -214,6 +214,89 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreAr
   }
 }
 
+// The common case of the above (no rotation, heads of up to 128 in multiples of 4, at most 8 NB query and key heads, float
+// weights): a warp's heads in one batch, and every load is asked for before the first is used; biases and weights, which no
+// kernel of a step writes, even before the wait for the kernel in front.
+template <typename A, int NB>
+__global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_small_kernel(QkStoreArgs p) {
+  __shared__ float red[2][QKS_WARPS];
+  pdl_launch_dependents();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, j = (threadIdx.x & 31) * 4;
+  const int H = p.H, heads = p.H + p.G, hd = p.hd, QW = H * hd, KW = p.G * hd, VW = p.G * p.vd;
+  const bool on = j < hd;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 b[NB], w[NB], x[NB];
+#pragma unroll
+  for (int n = 0; n < NB; n++) {
+    const int head = warp + n * QKS_WARPS;
+    const bool ok = on && head < heads;
+    const float* wp = (const float*)(head < H ? p.qw : p.kw);
+    b[n] = ok && p.bias ? *(const float4*)(p.bias + head * hd + j) : zero;
+    w[n] = ok && wp ? *(const float4*)(wp + (p.per_head ? j : head < H ? head * hd + j : head * hd - QW + j)) : zero;
+  }
+  const int e = threadIdx.x * 4;
+  float4 vb = p.bias && e < VW ? *(const float4*)(p.bias + QW + KW + e) : zero;
+  pdl_wait();
+  const int pos = p.tok_pos[t];
+  const A* c = (const A*)p.c + (size_t)t * p.ld;
+  A* vm = (A*)p.vmix + (size_t)t * VW;
+#pragma unroll
+  for (int n = 0; n < NB; n++) x[n] = on && warp + n * QKS_WARPS < heads ? ld4(c + (warp + n * QKS_WARPS) * hd + j) : zero;
+  float4 v = e < VW ? ld4(c + QW + KW + e) : zero, f = p.mix_mode == 2 && e < VW ? ld4((const A*)vm + e) : zero;
+  size_t page_slot = 0;
+  if (p.G > 0) {
+    const int page = p.block_table[(size_t)p.tok_seq[t] * p.max_pages + pos / SLLM_PAGE];
+    page_slot = (size_t)page * p.G * SLLM_PAGE + (pos % SLLM_PAGE);
+  }
+  float ss[NB];
+#pragma unroll
+  for (int n = 0; n < NB; n++) {
+    x[n].x += b[n].x; x[n].y += b[n].y; x[n].z += b[n].z; x[n].w += b[n].w;
+    ss[n] = warp_sum(fmaf(x[n].x, x[n].x, fmaf(x[n].y, x[n].y, fmaf(x[n].z, x[n].z, x[n].w * x[n].w))));
+  }
+  float rq = 1.f, rk = 1.f;
+  if (!p.per_head && (p.qw || p.kw)) {
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int n = 0; n < NB; n++) {
+      if (warp + n * QKS_WARPS < H) sq += ss[n]; else sk += ss[n];
+    }
+    if (j == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < QKS_WARPS; i++) { sq += red[0][i]; sk += red[1][i]; }
+    rq = 1.0f / sqrtf(sq / (float)QW + p.eps);
+    rk = 1.0f / sqrtf(sk / (float)(KW > 0 ? KW : 1) + p.eps);
+  }
+#pragma unroll
+  for (int n = 0; n < NB; n++) {
+    const int head = warp + n * QKS_WARPS;
+    if (head < heads && on) {
+      if (head < H ? p.qw != nullptr : p.kw != nullptr) {
+        const float r = p.per_head ? 1.0f / sqrtf(ss[n] / (float)hd + p.eps) : head < H ? rq : rk;
+        x[n] = make_float4(x[n].x * r * w[n].x, x[n].y * r * w[n].y, x[n].z * r * w[n].z, x[n].w * r * w[n].w);
+      }
+      if (head < H) st4((A*)p.q_out + (size_t)t * p.ldq + head * hd + j, x[n]);
+      else st4((A*)p.kpages + (page_slot + (size_t)(head - H) * SLLM_PAGE) * hd + j, x[n]);
+    }
+  }
+  for (int k = e; k < VW; k += QKS_WARPS * 32 * 4) {
+    if (k != e) {
+      v = ld4(c + QW + KW + k);
+      if (p.bias) vb = *(const float4*)(p.bias + QW + KW + k);
+      if (p.mix_mode == 2) f = ld4((const A*)vm + k);
+    }
+    v.x += vb.x; v.y += vb.y; v.z += vb.z; v.w += vb.w;
+    if (p.mix_mode == 1) st4(vm + k, v);
+    if (p.mix_mode == 2) {
+      const float a = 1.0f - p.lam;
+      v = make_float4(a * v.x + p.lam * f.x, a * v.y + p.lam * f.y, a * v.z + p.lam * f.z, a * v.w + p.lam * f.w);
+    }
+    st4((A*)p.vpages + (page_slot + (size_t)(k / p.vd) * SLLM_PAGE) * p.vd + k % p.vd, v);
+  }
+}
+
 // ------------------------------------------------------------------ convolution, norm, rotation, cache write
 // The same as qk_norm_store behind a short causal convolution, one block a token and the row never leaving the
 // chip: row t of y (A, row stride ldy) is the projection [queries | keys | values] of C = (H + G) hd + G vd

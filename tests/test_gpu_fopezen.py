@@ -452,7 +452,8 @@ def test_decode_splits_of_any_number_give_the_same():
 # --------------------------------------------------------------------------- the small kernels
 @pytest.mark.parametrize("H,G,hd,vd,rot,interleaved", [(4, 2, 12, 8, 0, False), (3, 1, 7, 5, 0, False), (5, 5, 64, 16, 16, False),
                                                        (2, 1, 9, 3, 4, True), (6, 2, 128, 64, 128, True), (2, 2, 512, 260, 0, False),
-                                                       (2, 1, 300, 8, 20, False)])
+                                                       (2, 1, 300, 8, 20, False), (20, 4, 128, 64, 0, False), (36, 9, 24, 40, 0, False),
+                                                       (60, 4, 8, 8, 0, False)])
 def test_the_store_kernel_adds_biases_norms_turns_mixes_and_fills_the_cache(H, G, hd, vd, rot, interleaved):
     from scriptling_llm_lib_b200.csrc.bindings import KernelSet
     g = torch.Generator().manual_seed(H + hd)
