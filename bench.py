@@ -1182,8 +1182,8 @@ def tufazen_kernels_alone(args):
             n_split = ks.decode.attention_splits(B, H, G, D, pages, sms)
             scratch = torch.empty(B * H * n_split * (D + 2), dtype=torch.float32, device=dev)
             tickets = torch.zeros(B * G, dtype=torch.int32, device=dev)
-            us = timed(lambda i: ks.decode.attn_decode_capped(q, o, c.seq_pos0, table, kp, vp, scratch, tickets, B, H, G, D, 0, D ** -0.5,
-                                                              n_split, 30.0, sink), 1)
+            us = timed(lambda i: ks.decode.attn_decode_general(q, o, c.seq_pos0, table, kp, vp, scratch, tickets, B, H, G, D, D, 0, D ** -0.5,
+                                                               n_split, softcap=30.0, sink=sink), 1)
             report(f"attn_decode {H}/{G} heads of {D}, cap and sinks, {n_split} splits ({label})", T, us, nbytes=B * ctxlen * G * 2 * D * esz)
             us = timed(lambda i: ks.decode.attn_decode(q, o, c.seq_pos0, table, kp, vp, scratch, B, H, G, D, 0, D ** -0.5, n_split,
                                                        tickets=tickets), 1)

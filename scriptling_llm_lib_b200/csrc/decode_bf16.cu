@@ -1070,7 +1070,6 @@ static int attn_decode_launch(const AttnDecodeArgs& a, bf16* out, int B, cudaStr
                               HD, a.n_split, a.sink);
     }
   }
-  if (a.softcap > 0.f || a.sink != nullptr) return SLLM_ERR_ARG;      // capped scores and sinks: the tensor-core kernel only
   if (a.cs != nullptr) {
     if (nrep % 4 == 0) e = sllm_launch(attn_decode_split_kernel<HD, 4, true, false>, grid, dim3(AD_WARPS * 32), 0, stream, a);
     else if (nrep % 2 == 0) e = sllm_launch(attn_decode_split_kernel<HD, 2, true, false>, grid, dim3(AD_WARPS * 32), 0, stream, a);
@@ -1095,8 +1094,7 @@ SLLM_EXPORT long long sllm_attn_decode_scratch_bytes(int B, int H, int hd, int n
 static int attn_decode_dispatch(const void* q, int q_ld, void* out, const int* seq_pos0, const int* block_table,
                                 int max_pages, const void* kpages, const void* vpages, void* scratch, int* tickets, int B,
                                 int H, int G, int hd, int window, float scale, int n_split, cudaStream_t stream,
-                                const void* cos_sin = nullptr, int rot = 0, int interleaved = 0, int write_kv = 0,
-                                float softcap = 0.f, const float* sink = nullptr) {
+                                const void* cos_sin = nullptr, int rot = 0, int interleaved = 0, int write_kv = 0) {
   if (B <= 0) return 0;
   if (G < 1 || H % G != 0 || n_split < 1 || (q_ld & 7) || ((uintptr_t)q & 15)) return SLLM_ERR_ARG;
   if (cos_sin != nullptr && (rot < 2 || rot > hd || (rot % (interleaved ? 8 : 16)) != 0 || tickets == nullptr)) return SLLM_ERR_ARG;
@@ -1105,8 +1103,6 @@ static int attn_decode_dispatch(const void* q, int q_ld, void* out, const int* s
                    write_kv, 0, 0.f, nullptr, hd, hd, 0, nullptr, 0};
   static const int late = getenv("SLLM_DECODE_LATE_KEYS") != nullptr;   // for comparisons
   a.late = late;
-  a.softcap = softcap;
-  a.sink = sink;
   switch (hd) {
     case 16: return attn_decode_launch<16>(a, (bf16*)out, B, stream);
     case 32: return attn_decode_launch<32>(a, (bf16*)out, B, stream);
@@ -1134,18 +1130,6 @@ SLLM_EXPORT int sllm_attn_decode_merged_bf16(const void* q, int q_ld, void* out,
   if (tickets == nullptr) return SLLM_ERR_ARG;
   return attn_decode_dispatch(q, q_ld, out, seq_pos0, block_table, max_pages, kpages, vpages, scratch, tickets, B, H, G, hd,
                               window, scale, n_split, stream);
-}
-
-// The same with capped scores and a sink per head (either may be off: softcap <= 0, sink null): for shapes the tensor-core
-// kernel serves (sllm_attn_decode_uses_mma); others are refused.
-SLLM_EXPORT int sllm_attn_decode_capped_bf16(const void* q, int q_ld, void* out, const int* seq_pos0,
-                                             const int* block_table, int max_pages, const void* kpages,
-                                             const void* vpages, void* scratch, int* tickets, int B, int H, int G, int hd,
-                                             int window, float scale, int n_split, float softcap, const float* sink,
-                                             cudaStream_t stream) {
-  if (tickets == nullptr || !attn_decode_uses_mma(B, H, G, hd) || getenv("SLLM_DECODE_SCALAR") != nullptr) return SLLM_ERR_ARG;
-  return attn_decode_dispatch(q, q_ld, out, seq_pos0, block_table, max_pages, kpages, vpages, scratch, tickets, B, H, G, hd,
-                              window, scale, n_split, stream, nullptr, 0, 0, 0, softcap, sink);
 }
 
 // The general form on the tensor-core kernel: keys hd wide and values vd wide (multiples of 8 up to 256 and 128), any number of

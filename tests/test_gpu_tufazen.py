@@ -606,13 +606,13 @@ def test_the_tensor_core_attention_kernels_with_a_cap_and_a_sink(H, G, hd, cap):
                                  torch.tensor([640], dtype=torch.int32).cuda(), bt, kpd, vpd, 1, 160, H, G, hd, 0, scale, err, cap, sd)
     assert float((out2.cpu().double()[[0, 158, 159]] - want[[12, 13, 14]]).abs().max()) < 2e-2
     dec = ks.decode
-    if dec.uses_tensor_cores(1, H, G, hd):
+    if dec.general_takes(hd, hd):
         for n_split in (1, 3, 6, 12):                 # more than eight splits are merged a warp a head
             out1 = torch.zeros(1, H * hd, dtype=torch.bfloat16, device="cuda")
             scratch = torch.empty(H * n_split * (hd + 2), dtype=torch.float32, device="cuda")
             tickets = torch.zeros(64, dtype=torch.int32, device="cuda")
-            dec.attn_decode_capped(qd[L - 1:].contiguous(), out1, torch.tensor([L - 1], dtype=torch.int32).cuda(), bt, kpd, vpd, scratch,
-                                   tickets, 1, H, G, hd, 0, scale, n_split, cap, sd)
+            dec.attn_decode_general(qd[L - 1:].contiguous(), out1, torch.tensor([L - 1], dtype=torch.int32).cuda(), bt, kpd, vpd, scratch,
+                                   tickets, 1, H, G, hd, hd, 0, scale, n_split, softcap=cap, sink=sd)
             assert float((out1.cpu().double() - want[-1:]).abs().max()) < 2e-2, n_split
             assert int(tickets.abs().sum()) == 0
 
