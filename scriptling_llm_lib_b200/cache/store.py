@@ -38,6 +38,8 @@ class KVGroup:
     k: torch.Tensor            # [len(units), n_pages, kv_heads, PAGE, head_dim]
     v: torch.Tensor
     pages: dict[int, list[int]] = field(default_factory=dict)   # slot -> page id per page index (-1: given back)
+    behind: dict[int, int] = field(default_factory=dict)        # slot -> page indices below this one are settled: given back or kept
+    table: np.ndarray | None = None    # [slots, pages so far] int32: the same ids as `pages` (-1: none), a step's block tables are cut from it
 
     def unit_storage(self, unit: int):
         i = self.units.index(unit)
@@ -48,8 +50,18 @@ class KVGroup:
 
     def grow(self, slot: int, new_len: int) -> None:
         lst = self.pages[slot]
-        while len(lst) < pages_for(new_len):
-            lst.append(self.pool.alloc())
+        n = pages_for(new_len)
+        if n > self.table.shape[1]:
+            more = np.full((self.table.shape[0], max(n, 2 * self.table.shape[1]) - self.table.shape[1]), -1, dtype=np.int32)
+            self.table = np.concatenate([self.table, more], axis=1)
+        while len(lst) < n:
+            page = self.pool.alloc()
+            self.table[slot, len(lst)] = page
+            lst.append(page)
+
+    def open(self, slot: int) -> None:
+        self.pages[slot] = []
+        self.behind[slot] = pages_for(self.need.keep)
 
     def release_unseen(self, slot: int, length: int) -> None:
         """Give back the pages no query at a position >= length can see (the need's kind says which; pages that hold one of
@@ -57,16 +69,20 @@ class KVGroup:
         first_seen = self.need.first_needed(length)
         if first_seen <= 0:
             return
-        lst = self.pages[slot]
-        for i, pg in enumerate(lst):
-            if pg >= 0 and (i + 1) * PAGE - 1 < first_seen and i * PAGE >= self.need.keep:
-                self.pool.free(pg)
-                lst[i] = -1
+        lst, i = self.pages[slot], self.behind[slot]
+        while i < len(lst) and (i + 1) * PAGE - 1 < first_seen:
+            self.pool.free(lst[i])
+            lst[i] = self.table[slot, i] = -1
+            i += 1
+        self.behind[slot] = i
 
     def release_all(self, slot: int) -> None:
-        for pg in self.pages.pop(slot):
+        lst = self.pages.pop(slot)
+        for pg in lst:
             if pg >= 0:
                 self.pool.free(pg)
+        self.table[slot, :len(lst)] = -1
+        del self.behind[slot]
 
 
 class SequenceCache:
@@ -90,7 +106,8 @@ class SequenceCache:
             shape = (len(units), n_pages + 1, need.kv_heads, PAGE, need.head_dim)
             v_shape = shape[:-1] + (need.value_dim,)
             g = KVGroup(need, units, FreeList(n_pages, f"cache page ({need.kind})"),
-                        torch.empty(shape, dtype=dtype, device=device), torch.empty(v_shape, dtype=dtype, device=device))
+                        torch.empty(shape, dtype=dtype, device=device), torch.empty(v_shape, dtype=dtype, device=device),
+                        table=np.full((n_slots, 16), -1, dtype=np.int32))
             for u in units:
                 self.group_of_unit[u] = len(self.groups)
             self.groups.append(g)
@@ -110,7 +127,7 @@ class SequenceCache:
         slot = self.slots.alloc()
         self.length[slot] = 0
         for g in self.groups:
-            g.pages[slot] = []
+            g.open(slot)
         def zero(st):
             if isinstance(st, dict):
                 for t in st.values():
@@ -161,10 +178,10 @@ class SequenceCache:
     def block_table(self, group: int, slots: list[int], width: int | None = None) -> np.ndarray:
         g = self.groups[group]
         w = max(1, max(len(g.pages[s]) for s in slots)) if width is None else width
+        if w <= g.table.shape[1]:
+            return g.table[slots, :w]
         bt = np.full((len(slots), w), -1, dtype=np.int32)
-        for i, s in enumerate(slots):
-            lst = g.pages[s]
-            bt[i, :len(lst)] = lst
+        bt[:, :g.table.shape[1]] = g.table[slots]
         return bt
 
     def tokens_capacity(self) -> int:
