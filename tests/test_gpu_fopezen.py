@@ -368,7 +368,7 @@ def attend_rows(q, k, v, rows, H, G, scale, window, keep, sink):
     (4, 2, 64, 64, 100, 3, 400, True, True, "bfloat16"), (4, 4, 64, 64, 64, 64, 300, False, False, "bfloat16"),
     (6, 2, 128, 128, 40, 70, 390, True, True, "bfloat16"), (4, 2, 128, 128, 200, 1, 500, False, True, "bfloat16"),
     (3, 3, 128, 128, 33, 5, 385, True, False, "bfloat16"), (3, 1, 128, 128, 300, 129, 513, True, True, "bfloat16"),
-    (8, 2, 96, 32, 136, 17, 420, True, True, "bfloat16"), (12, 1, 72, 24, 50, 140, 330, False, True, "bfloat16"),
+    (6, 3, 88, 32, 120, 17, 420, True, True, "bfloat16"), (12, 1, 72, 24, 50, 140, 330, False, True, "bfloat16"),
     (2, 2, 256, 128, 64, 63, 260, True, False, "bfloat16"), (4, 1, 40, 104, 65, 65, 270, True, True, "bfloat16"),
     (4, 2, 8, 8, 20, 2, 150, True, True, "bfloat16"), (4, 2, 128, 64, None, 0, 300, True, True, "bfloat16"),
     (4, 2, 128, 128, None, 0, 300, False, True, "bfloat16"), (3, 1, 6, 10, 30, 4, 200, True, False, "bfloat16"),
