@@ -89,23 +89,28 @@ class KernelSet:
         return fn
 
     # ------------------------------------------------------------------ embedding
-    def embed_rows(self, ids, table, out, err_flag):
+    def embed_rows(self, ids, table, out, err_flag, scale=1.0, copy=None):
+        """out float32 [T, d] = scale * table[ids[t]]; `copy` (float32 [T, d]) receives the same."""
         T, d = out.shape
+        if copy is not None and tuple(copy.shape) != (T, d):
+            raise KernelError(f"embed_rows: a copy of {tuple(copy.shape)} for rows of {(T, d)}")
         _check(self._fn("embed_rows")(_ptr(ids, torch.int32, "ids"), _ptr(table, self.dtype, "table"),
-                                      _ptr(out, torch.float32, "out"), c_int(T), c_int(d), c_int(table.shape[0]),
-                                      _ptr(err_flag, torch.int32, "err"), _stream()), "embed_rows")
+                                      _ptr(out, torch.float32, "out"), _ptr(copy, torch.float32, "copy"), c_float(scale),
+                                      c_int(T), c_int(d), c_int(table.shape[0]), _ptr(err_flag, torch.int32, "err"), _stream()), "embed_rows")
 
-    def embed_pair_rows(self, ids, ctx, table, pair_table, buckets, mul_prev, mul_cur, last, out, err_flag):
-        """out float32 [T, d] = table[ids[t]] + pair_table[(previous token * mul_prev + ids[t] * mul_cur) mod buckets], the
-        pair table's row `buckets` for a sequence's first token; `last` int32 [slots]: the sequences' last tokens (read, then set)."""
+    def embed_pair_rows(self, ids, ctx, table, pair_table, buckets, mul_prev, mul_cur, last, out, err_flag, scale=1.0, copy=None):
+        """out float32 [T, d] = scale * table[ids[t]] + pair_table[(previous token * mul_prev + ids[t] * mul_cur) mod buckets], the
+        pair table's row `buckets` for a sequence's first token; `last` int32 [slots]: the sequences' last tokens (read, then set);
+        `copy` (float32 [T, d]) receives what out does."""
         T, d = out.shape
-        if tuple(pair_table.shape) != (buckets + 1, d) or table.shape[1] != d or last.dim() != 1:
+        if (tuple(pair_table.shape) != (buckets + 1, d) or table.shape[1] != d or last.dim() != 1
+                or (copy is not None and tuple(copy.shape) != (T, d))):
             raise KernelError(f"embed_pair_rows shapes: table {tuple(table.shape)}, pair table {tuple(pair_table.shape)}, buckets {buckets}")
         _check(self._fn("embed_pair_rows")(_ptr(ids, torch.int32, "ids"), _ptr(ctx.tok_pos, torch.int32, "tok_pos"),
                                            _ptr(ctx.tok_seq, torch.int32, "tok_seq"), _ptr(ctx.seq_start, torch.int32, "seq_start"),
                                            _ptr(ctx.slots, torch.int32, "slots"), _ptr(table, self.dtype, "table"),
-                                           _ptr(pair_table, self.dtype, "pair_table"), _ptr(out, torch.float32, "out"), c_int(T), c_int(d),
-                                           c_int(table.shape[0]), c_int(buckets), c_longlong(mul_prev), c_longlong(mul_cur),
+                                           _ptr(pair_table, self.dtype, "pair_table"), _ptr(out, torch.float32, "out"),
+                                           _ptr(copy, torch.float32, "copy"), c_float(scale), c_int(T), c_int(d), c_int(table.shape[0]), c_int(buckets), c_longlong(mul_prev), c_longlong(mul_cur),
                                            _ptr(last, torch.int32, "last"), _ptr(err_flag, torch.int32, "err"), _stream()),
                "embed_pair_rows")
 
@@ -276,6 +281,13 @@ class KernelSet:
         if getattr(self, "_mix", None) is None:
             self._mix = MixKernels(self.dtype)
         return self._mix
+
+    @property
+    def ssd(self) -> "SsdKernels":
+        """The state-space recurrence with one decay per head and token (its own library, compiled and loaded on first use)."""
+        if getattr(self, "_ssd", None) is None:
+            self._ssd = SsdKernels(self.dtype)
+        return self._ssd
 
     @property
     def gate(self) -> "GateKernels":
@@ -977,15 +989,16 @@ class MixKernels:
                                          c_int(block_table.shape[1]), _ptr(dense, self.dtype, "dense"), c_int(dense.shape[0]),
                                          c_int(dense.shape[1]), _stream()), "latent_gather")
 
-    def latent_heads(self, q, kv, dense, rank, ctx, table, kt, vt, qt, n_heads, dim, rot_dim, v_dim, hd):
-        """Keys [Wuk c | rotated part | 0], values [Wuv c | 0] and queries [q | 0] per head, `hd` wide, keys and values
-        into pages of their own by `table` (a prompt step from position 0)."""
+    def latent_heads(self, q, kv, dense, rank, ctx, table, kt, vt, qt, n_heads, dim, rot_dim, v_dim):
+        """Keys [Wuk c | rotated part | 0] and values [Wuv c | 0] per head, as wide as kt's and vt's rows, into pages of their
+        own by `table` (a prompt step from position 0), and queries [q | 0] as wide as the keys into qt (None: they stay)."""
         _check(self._fn("latent_heads")(self._view(q, "q"), c_int(q.stride(0)), self._view(kv, "kv"), c_int(kv.stride(0)),
                                         self._view(dense, "dense"), c_int(dense.stride(0)), c_int(rank),
                                         _ptr(ctx.tok_pos, torch.int32, "tok_pos"), _ptr(ctx.tok_seq, torch.int32, "tok_seq"),
                                         _ptr(table, torch.int32, "table"), c_int(table.shape[1]), _ptr(kt, self.dtype, "kt"),
-                                        _ptr(vt, self.dtype, "vt"), _ptr(qt, self.dtype, "qt"), c_int(q.shape[0]), c_int(n_heads),
-                                        c_int(dim), c_int(rot_dim), c_int(v_dim), c_int(hd), _stream()), "latent_heads")
+                                        _ptr(vt, self.dtype, "vt"), _ptr(qt, self.dtype if qt is not None else None, "qt"),
+                                        c_int(q.shape[0]), c_int(n_heads), c_int(dim), c_int(rot_dim), c_int(v_dim), c_int(kt.shape[-1]),
+                                        c_int(vt.shape[-1]), _stream()), "latent_heads")
 
     def latent_absorb(self, q, wuk, qa, n_heads, dim, rot_dim, rank, scale):
         """qa float32 [T, H, rank + rot_dim] = scale * [Wuk_h^T q_h[:dim] | q_h[dim:]] for every head."""
@@ -995,19 +1008,28 @@ class MixKernels:
                                          _ptr(qa, torch.float32, "qa"), c_int(q.shape[0]), c_int(n_heads), c_int(dim),
                                          c_int(rot_dim), c_int(rank), c_float(scale), _stream()), "latent_absorb")
 
-    def latent_attn(self, qa, pages, ctx, block_table, part, n_heads, rank, rot_dim, n_split):
+    def latent_attn(self, qa, pages, ctx, block_table, part, n_heads, rank, rot_dim, n_split, window=0):
+        """`window` > 0: a row sees its own position and the window - 1 before it; 0: every earlier one."""
         _check(self._fn("latent_attn")(
             _ptr(qa, torch.float32, "qa"), _ptr(pages, self.dtype, "pages"), _ptr(ctx.tok_pos, torch.int32, "tok_pos"),
             _ptr(ctx.tok_seq, torch.int32, "tok_seq"), _ptr(block_table, torch.int32, "block_table"), c_int(block_table.shape[1]),
             _ptr(part, torch.float32, "part"), c_int(qa.shape[0]), c_int(n_heads), c_int(rank), c_int(rot_dim), c_int(n_split),
-            _stream()), "latent_attn")
+            c_int(window), _stream()), "latent_attn")
 
-    def latent_expand(self, part, olat, wuv, out, n_heads, v_dim, rank, n_split):
-        """Merges the splits of `part` into olat float32 [T, H, rank] (scratch), then out[t, h] = Wuv_h olat[t, h]."""
+    def latent_expand(self, part, olat, wuv, out, n_heads, v_dim, rank, n_split, sink=None, gate=None):
+        """Merges the splits of `part` into olat float32 [T, H, rank] (scratch), then out[t, h] = Wuv_h olat[t, h]. `sink` float32
+        [H]: exp(sink) joins the head's denominator once; `gate` (a column slice, element type): logits [T, H] or [T, H V]
+        whose sigmoid multiplies the head or the element."""
+        mode = 0
+        if gate is not None:
+            mode = 1 if gate.shape[1] == n_heads else 2
+            if gate.dtype != self.dtype or tuple(gate.shape) != (out.shape[0], n_heads * (v_dim if mode == 2 else 1)):
+                raise KernelError(f"latent_expand: gate logits {tuple(gate.shape)} {gate.dtype} for {n_heads} heads of {v_dim}")
         _check(self._fn("latent_expand")(_ptr(part, torch.float32, "part"), _ptr(olat, torch.float32, "olat"),
                                          _ptr(wuv, self.dtype, "wuv"), _ptr(out, self.dtype, "out"), c_int(out.shape[1]),
-                                         c_int(out.shape[0]), c_int(n_heads), c_int(v_dim), c_int(rank), c_int(n_split), _stream()),
-               "latent_expand")
+                                         c_int(out.shape[0]), c_int(n_heads), c_int(v_dim), c_int(rank), c_int(n_split),
+                                         _ptr(sink, torch.float32, "sink"), self._view(gate, "gate") if gate is not None else c_void_p(0),
+                                         c_int(gate.stride(0) if gate is not None else 0), c_int(mode), _stream()), "latent_expand")
         LAUNCHES[0] += 1
 
     def selective_scan(self, x, dt_raw, dt_bias, a_log, dskip, bc, b_col, c_col, z, state, ctx, out, inner, n_state):
@@ -1106,6 +1128,62 @@ class MixKernels:
                                        c_int(out.shape[1]), _stream()), "moe_combine")
 
 
+class SsdKernels:
+    """Launchers of ssd_kernels.cuh: the state-space recurrence with one decay per head and token, and the norm over equal
+    runs of columns behind it. `dtype` is the element type of activations; step sizes, decays, state and sums are float32."""
+    CHUNK, CHUNK_MIN_ROWS, CHUNK_MAX_STATE = 128, 64, 256
+
+    def __init__(self, dtype: torch.dtype):
+        if dtype not in _SUFFIX:
+            raise KernelError(f"no kernels for {dtype}; supported: float32, bfloat16")
+        self.dtype, self.suffix = dtype, _SUFFIX[dtype]
+        self.lib = load_library("ssd_" + self.suffix)
+        self._fns: dict[str, object] = {}
+
+    _fn = SequenceKernels._fn
+    _view = staticmethod(SequenceKernels._view)
+
+    def scan(self, xbc, dt, dt_bias, a_log, dskip, z, state, ctx, out, n_heads, n_groups, head_dim, n_state, weight=None, chunked=None):
+        """xbc [T, H V + 2 G N] (x | B | C), dt [T, H] raw step sizes, z [T, H V]: views of the element type; dt_bias, a_log,
+        dskip float32 [H]; state float32 [slots, H, N, V] (read and advanced); out [T, H V] = y * silu(z). With `weight`
+        (float32 [H V]) out is also multiplied by it, and the answer is float32 [parts, T]: partial sums of (y silu(z))^2 over a
+        row. `chunked`: through the tensor cores in chunks of rows (None: where a bfloat16 run is long enough)."""
+        T, HV = out.shape
+        if (HV != n_heads * head_dim or tuple(xbc.shape) != (T, HV + 2 * n_groups * n_state) or tuple(dt.shape) != (T, n_heads)
+                or tuple(z.shape) != (T, HV) or tuple(state.shape[1:]) != (n_heads, n_state, head_dim)):
+            raise KernelError(f"ssd shapes: xbc {tuple(xbc.shape)}, dt {tuple(dt.shape)}, z {tuple(z.shape)}, state {tuple(state.shape)}")
+        for t, name in ((xbc, "xbc"), (dt, "dt"), (z, "z"), (out, "out")):
+            if t.dtype != self.dtype:
+                raise KernelError(f"ssd: {name} has dtype {t.dtype}, expected {self.dtype}")
+        if chunked is None:
+            chunked = self.dtype == torch.bfloat16 and ctx.max_new >= self.CHUNK_MIN_ROWS
+        chunked = chunked and n_state <= self.CHUNK_MAX_STATE
+        states = decays = sumsq = None
+        if chunked:
+            n = T // self.CHUNK + ctx.n_seqs
+            states = torch.empty((n, n_heads, n_state, head_dim), dtype=torch.float32, device=out.device)
+            decays = torch.empty((n, n_heads), dtype=torch.float32, device=out.device)
+        if weight is not None:
+            sumsq = torch.empty((n_heads * -(-head_dim // (64 if chunked else 32)), T), dtype=torch.float32, device=out.device)
+        _check(self._fn("ssd")(
+            self._view(xbc, "xbc"), c_int(xbc.stride(0)), self._view(dt, "dt"), c_int(dt.stride(0)), _ptr(dt_bias, torch.float32, "dt_bias"),
+            _ptr(a_log, torch.float32, "a_log"), _ptr(dskip, torch.float32, "dskip"), self._view(z, "z"), c_int(z.stride(0)),
+            _ptr(state, torch.float32, "state"), _ptr(ctx.seq_start, torch.int32, "seq_start"), _ptr(ctx.slots, torch.int32, "slots"),
+            self._view(out, "out"), c_int(out.stride(0)), _ptr(weight, torch.float32, "weight"), _ptr(sumsq, torch.float32, "sumsq"),
+            _ptr(states, torch.float32, "states"), _ptr(decays, torch.float32, "decays"), c_int(ctx.n_seqs), c_int(max(1, ctx.max_new)),
+            c_int(T), c_int(n_heads), c_int(n_groups), c_int(head_dim), c_int(n_state), _stream()), "ssd")
+        if chunked:
+            LAUNCHES[0] += 2
+        return sumsq
+
+    def group_norm(self, u, weight, y, groups, eps):
+        """y [T, W] = u, every one of `groups` equal runs of columns over its own root mean square, times weight (float32 [W])."""
+        if tuple(u.shape) != tuple(y.shape) or weight.numel() != u.shape[1] or u.shape[1] % groups:
+            raise KernelError(f"group_norm shapes: u {tuple(u.shape)}, weight {tuple(weight.shape)}, {groups} groups")
+        _check(self._fn("group_norm")(_ptr(u, self.dtype, "u"), _ptr(weight, torch.float32, "weight"), _ptr(y, self.dtype, "y"),
+                                      c_int(u.shape[0]), c_int(u.shape[1]), c_int(groups), c_float(eps), _stream()), "group_norm")
+
+
 class GateKernels:
     """Launchers of gate_kernels.cuh. `dtype` is the element type of activations and weights; norms, gates,
     angles and the residual sum are float32 in both sets."""
@@ -1122,12 +1200,13 @@ class GateKernels:
     _view = staticmethod(SequenceKernels._view)
 
     def qk_norm_store(self, c, q_out, tok_pos, tok_seq, block_table, cos_sin, kpages, vpages, n_heads, n_kv, head_dim, v_dim,
-                      rot, interleaved, q_weight, k_weight, eps, bias=None, per_head=False, value_mix=None):
+                      rot, interleaved, q_weight, k_weight, eps, bias=None, per_head=False, value_mix=None, norm_after=False):
         """Row t of c (float32 or element type; a view) holds [queries | keys | values] of a token; `bias` (float32, the
         same columns) is added first. Queries and keys are each divided by the root mean square of their whole part
         (`per_head`: of every head by itself, weights of one head's width) and multiplied by q_weight / k_weight (None: as
         they are), turned by the table over their first `rot` dims, and go to q_out [T, n_heads * head_dim] and, with
-        the values, to the rows' places in the cache pages (n_kv == 0: queries only). `value_mix` = (kept, None): the values
+        the values, to the rows' places in the cache pages (n_kv == 0: queries only). `norm_after`: every head
+        is divided by its own root mean square after it has turned, without a weight. `value_mix` = (kept, None): the values
         also go to kept [T, n_kv * v_dim] (element type); (kept, lam): stored are (1 - lam) * values + lam * kept."""
         if bias is not None and bias.numel() != (n_heads + n_kv) * head_dim + n_kv * v_dim:
             raise KernelError(f"qk_norm_store: a bias of {bias.numel()} columns")
@@ -1152,7 +1231,8 @@ class GateKernels:
             _ptr(vpages, self.dtype if vpages is not None else None, "vpages"), c_int(c.shape[0]), c_int(n_heads), c_int(n_kv),
             c_int(head_dim), c_int(v_dim), c_int(rot), c_int(1 if interleaved else 0), _ptr(q_weight, None, "q_weight"),
             _ptr(k_weight, None, "k_weight"), c_int(w_f32), c_int(1 if per_head else 0), c_float(eps),
-            _ptr(kept, self.dtype if kept is not None else None, "kept"), c_int(mode), c_float(lam), _stream()), "qk_norm_store")
+            _ptr(kept, self.dtype if kept is not None else None, "kept"), c_int(mode), c_float(lam), c_int(1 if norm_after else 0),
+            _stream()), "qk_norm_store")
 
     FUSED_CONV_MAX_WIDTH = 200 * 1024 // 4      # the row stays in shared memory as floats
 

@@ -1,5 +1,6 @@
 // Kernels around gated mixers and gated side inputs, for float and bfloat16 activations (A):
-//   qk_norm_store    biases of the projections, RMS norm of queries and keys (per head, or over all heads at once),
+//   qk_norm_store    biases of the projections, RMS norm of queries and keys (per head or over all heads, before they turn,
+//                    or per head after),
 //                    rotation by position, values mixed with an earlier layer's, queries out, keys and values into
 //                    the paged cache
 //   head_gate        attention output of every head times the sigmoid of that head's gate logit
@@ -27,7 +28,8 @@ __device__ __forceinline__ float gelu_tanh_f(float v) {
 // keys are divided by their root mean square and multiplied by the weight: over ALL the columns of the query part and of
 // the key part (weights of H * hd and G * hd), or with `per_head` over every head by itself (weights of hd, shared by the
 // heads). Then the first `rot` dims of every query and key head turn by the token's position (table cs[pos][i] = (cos, sin);
-// half pairing i with i + rot / 2, or adjacent pairs), queries go to q_out [T, ldq], keys and values to the token's place in
+// half pairing i with i + rot / 2, or adjacent pairs). With `norm_after` every query and key head is instead divided by its
+// root mean square once it has turned, without a weight (qw and kw null). Queries go to q_out [T, ldq], keys and values to the token's place in
 // the cache pages. Values may be mixed on the way with those an earlier layer projected for the same token, kept in vmix
 // [T, G * vd]: mix_mode 1 writes them there, mode 2 stores (1 - lam) * v + lam * vmix. G == 0: queries only.
 struct QkStoreArgs {
@@ -40,6 +42,7 @@ struct QkStoreArgs {
   int H, G, hd, vd, rot, interleaved;
   const void* qw; const void* kw; int w_f32; int per_head; float eps;
   void* vmix; int mix_mode; float lam;
+  int norm_after;
 };
 
 template <int V> struct Pack { float f[V]; };
@@ -164,6 +167,41 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreAr
       float r = is_q ? rq : rk;
       if (p.per_head && w) r = 1.0f / sqrtf(warp_sum(squares(n, head)) / (float)hd + p.eps);
       A* dst = is_q ? (A*)p.q_out + (size_t)t * p.ldq + col : (A*)p.kpages + (page_slot + (size_t)(head - H) * SLLM_PAGE) * hd;
+      if constexpr (V == 4) {
+        if (p.norm_after && (p.interleaved || p.rot == 0)) {             // a lane's four elements are two whole pairs: no exchange
+#pragma unroll
+          for (int it = 0; it < NIT; it++) {
+            const int j = (it * 32 + lane) * V;
+#pragma unroll
+            for (int i = 0; i < V; i += 2)
+              if (j + i < p.rot) {
+                const float2 a = csr[(j + i) >> 1];
+                const float x0 = x[n][it].f[i], x1 = x[n][it].f[i + 1];
+                x[n][it].f[i] = x0 * a.x - x1 * a.y;
+                x[n][it].f[i + 1] = x1 * a.x + x0 * a.y;
+              }
+          }
+          r = 1.0f / sqrtf(warp_sum(squares(n, head)) / (float)hd + p.eps);
+#pragma unroll
+          for (int it = 0; it < NIT; it++) {
+            const int j = (it * 32 + lane) * V;
+            if (j >= hd) break;
+#pragma unroll
+            for (int i = 0; i < V; i++) x[n][it].f[i] *= r;
+            st_pack<A, V>(dst + j, x[n][it]);
+          }
+          continue;
+        }
+      }
+      if (p.norm_after && p.rot == 0) {
+        r = 1.0f / sqrtf(warp_sum(squares(n, head)) / (float)hd + p.eps);
+#pragma unroll
+        for (int it = 0; it < NIT; it++)
+          if ((it * 32 + lane) * V < hd) {
+#pragma unroll
+            for (int i = 0; i < V; i++) x[n][it].f[i] *= r;
+          }
+      }
 #pragma unroll
       for (int it = 0; it < NIT; it++) {
         const int j = (it * 32 + lane) * V;
@@ -182,14 +220,26 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreAr
       }
       if (p.rot > 0) {                                                   // a lane turns a pair; the rest passes as it is
         __syncwarp();
+        float ra = 1.f;
+        if (p.norm_after) {                                              // the sum is over the turned head
+          float ss = 0.f;
+          for (int i = lane; i < half; i += 32) {
+            const int i0 = p.interleaved ? 2 * i : i, i1 = p.interleaved ? 2 * i + 1 : i + half;
+            const float2 a = csr[i];
+            const float x0 = wrow[i0], x1 = wrow[i1], y0 = x0 * a.x - x1 * a.y, y1 = x1 * a.x + x0 * a.y;
+            ss = fmaf(y0, y0, fmaf(y1, y1, ss));
+          }
+          for (int j = p.rot + lane; j < hd; j += 32) ss = fmaf(wrow[j], wrow[j], ss);
+          ra = 1.0f / sqrtf(warp_sum(ss) / (float)hd + p.eps);
+        }
         for (int i = lane; i < half; i += 32) {
           const int i0 = p.interleaved ? 2 * i : i, i1 = p.interleaved ? 2 * i + 1 : i + half;
           const float2 a = csr[i];
           const float x0 = wrow[i0], x1 = wrow[i1];
-          dst[i0] = from_f32<A>(x0 * a.x - x1 * a.y);
-          dst[i1] = from_f32<A>(x1 * a.x + x0 * a.y);
+          dst[i0] = from_f32<A>((x0 * a.x - x1 * a.y) * ra);
+          dst[i1] = from_f32<A>((x1 * a.x + x0 * a.y) * ra);
         }
-        for (int j = p.rot + lane; j < hd; j += 32) dst[j] = from_f32<A>(wrow[j]);
+        for (int j = p.rot + lane; j < hd; j += 32) dst[j] = from_f32<A>(wrow[j] * ra);
         __syncwarp();
       }
     }

@@ -12,11 +12,11 @@
 #include "common.cuh"
 
 // ------------------------------------------------------------------ embedding
-// out[t, :] = table[ids[t], :] widened to float (the residual stream is float in both paths).
-// An id outside the table writes zeros and raises *err (the host checks ids before it launches).
+// out[t, :] = scale * table[ids[t], :] in float (the residual stream is float in both paths); `copy` (or null) receives the
+// same rows once more, for a layer that adds them to the stream again later. An id outside the table writes zeros and raises *err (the host checks ids before it launches).
 template <typename W>
 __global__ void embed_rows_kernel(const int* __restrict__ ids, const W* __restrict__ table,
-                                  float* __restrict__ out, int d, int vocab, int* err) {
+                                  float* __restrict__ out, float* __restrict__ copy, float scale, int d, int vocab, int* err) {
   pdl_launch_dependents();
   pdl_wait();
   int t = blockIdx.x;
@@ -25,7 +25,11 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const W* __restri
   if (!ok && threadIdx.x == 0) atomicExch(err, 1);
   const W* src = table + (size_t)(ok ? id : 0) * d;
   float* dst = out + (size_t)t * d;
-  for (int j = threadIdx.x; j < d; j += blockDim.x) dst[j] = ok ? to_f32(src[j]) : 0.f;
+  for (int j = threadIdx.x; j < d; j += blockDim.x) {
+    const float v = ok ? to_f32(src[j]) * scale : 0.f;
+    dst[j] = v;
+    if (copy) copy[(size_t)t * d + j] = v;
+  }
 }
 
 // The embedding with a vector per position: out[t, 2i] = table[ids[t], 2i] + sin(pos f_i), out[t, 2i + 1] = ... + cos(pos f_i).
@@ -55,15 +59,15 @@ __global__ void embed_rows_sinusoid_kernel(const int* __restrict__ ids, const in
 }
 
 // The embedding with a second table looked up by the pair (previous token, token):
-// out[t, :] = table[ids[t], :] + pair_table[r, :], r = (prev * mul_prev + ids[t] * mul_cur) mod buckets, and r = buckets (the
+// out[t, :] = scale * table[ids[t], :] + pair_table[r, :] (and the same to `copy` where there is one), r = (prev * mul_prev + ids[t] * mul_cur) mod buckets, and r = buckets (the
 // table's last row) for a sequence's first token (tok_pos 0). The previous token of a step's row is the row before it; for
 // the first row of a sequence's run it is what `last` [slots] holds, the sequence's state, which the same block then sets to
 // the run's last token (one block reads and writes a sequence's entry, so runs of any length keep it in order).
 template <typename W>
 __global__ void embed_pair_rows_kernel(const int* __restrict__ ids, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                                        const int* __restrict__ seq_start, const int* __restrict__ slots, const W* __restrict__ table,
-                                       const W* __restrict__ pair_table, float* __restrict__ out, int d, int vocab, int buckets,
-                                       long long mul_prev, long long mul_cur, int* __restrict__ last, int* err) {
+                                       const W* __restrict__ pair_table, float* __restrict__ out, float* __restrict__ copy, float scale, int d,
+                                       int vocab, int buckets, long long mul_prev, long long mul_cur, int* __restrict__ last, int* err) {
   __shared__ int s_prev;
   int t = blockIdx.x;
   int id = ids[t];
@@ -86,7 +90,11 @@ __global__ void embed_pair_rows_kernel(const int* __restrict__ ids, const int* _
   const W* src = table + (size_t)(ok ? id : 0) * d;
   const W* src2 = pair_table + (size_t)(ok ? r : 0) * d;
   float* dst = out + (size_t)t * d;
-  for (int j = threadIdx.x; j < d; j += blockDim.x) dst[j] = ok ? to_f32(src[j]) + to_f32(src2[j]) : 0.f;
+  for (int j = threadIdx.x; j < d; j += blockDim.x) {
+    const float v = ok ? fmaf(to_f32(src[j]), scale, to_f32(src2[j])) : 0.f;
+    dst[j] = v;
+    if (copy) copy[(size_t)t * d + j] = v;
+  }
 }
 
 // ------------------------------------------------------------------ residual add + RMSNorm

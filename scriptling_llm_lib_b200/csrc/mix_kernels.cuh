@@ -445,24 +445,50 @@ __global__ void latent_gather_kernel(const A* __restrict__ pages, const int* __r
   for (int j = threadIdx.x; j < W; j += blockDim.x) dense[(size_t)t * W + j] = src[j];
 }
 
-// heads: keys and values per head for a prompt that starts at position 0, laid out as pages of their own so that an
-// attention kernel for keys and values of one width `hd` >= max(D + P, V) can run on them. kv[t] = [Wuk c | Wuv c] (H D
-// and H V wide), dense[t][R ..] the rotated key part. kt[page][h][place] = [key of head h | rotated part | 0 ..],
-// vt[...] = [value of head h | 0 ..], qt[t][h] = [query of head h (D + P) | 0 ..]; the page of (sequence, position) comes
-// from `table` [sequences][max_pages].
+// heads: keys and values per head for a prompt that starts at position 0, laid out as pages of their own so that the
+// attention kernels for per-head keys (`kw` >= D + P wide) and values (`vw` >= V wide) can run on them. kv[t] = [Wuk c |
+// Wuv c] (H D and H V wide), dense[t][R ..] the rotated key part. kt[page][h][place] = [key of head h | rotated part | 0 ..],
+// vt[...] = [value of head h | 0 ..], qt[t][h] = [query of head h (D + P) | 0 ..] (qt null: queries stay where they are);
+// the page of (sequence, position) comes from `table` [sequences][max_pages].
 template <typename A>
 __global__ void latent_heads_kernel(const A* __restrict__ q, int ldq, const A* __restrict__ kv, int ldkv,
                                     const A* __restrict__ dense, int ldd, int R, const int* __restrict__ tok_pos,
                                     const int* __restrict__ tok_seq, const int* __restrict__ table, int max_pages,
-                                    A* __restrict__ kt, A* __restrict__ vt, A* __restrict__ qt, int H, int D, int P, int V, int hd) {
+                                    A* __restrict__ kt, A* __restrict__ vt, A* __restrict__ qt, int H, int D, int P, int V, int kw, int vw) {
   int t = blockIdx.x, h = blockIdx.y;
   int pos = tok_pos[t];
-  size_t at = (((size_t)table[(size_t)tok_seq[t] * max_pages + pos / SLLM_PAGE] * H + h) * SLLM_PAGE + pos % SLLM_PAGE) * hd;
+  size_t at = ((size_t)table[(size_t)tok_seq[t] * max_pages + pos / SLLM_PAGE] * H + h) * SLLM_PAGE + pos % SLLM_PAGE;
   const A zero = from_f32<A>(0.f);
-  for (int j = threadIdx.x; j < hd; j += blockDim.x) {
-    kt[at + j] = j < D ? kv[(size_t)t * ldkv + (size_t)h * D + j] : (j < D + P ? dense[(size_t)t * ldd + R + j - D] : zero);
-    vt[at + j] = j < V ? kv[(size_t)t * ldkv + (size_t)H * D + (size_t)h * V + j] : zero;
-    qt[((size_t)t * H + h) * hd + j] = j < D + P ? q[(size_t)t * ldq + (size_t)h * (D + P) + j] : zero;
+  for (int j = threadIdx.x; j < kw; j += blockDim.x) {
+    kt[at * kw + j] = j < D ? kv[(size_t)t * ldkv + (size_t)h * D + j] : (j < D + P ? dense[(size_t)t * ldd + R + j - D] : zero);
+    if (qt) qt[((size_t)t * H + h) * kw + j] = j < D + P ? q[(size_t)t * ldq + (size_t)h * (D + P) + j] : zero;
+  }
+  for (int j = threadIdx.x; j < vw; j += blockDim.x)
+    vt[at * vw + j] = j < V ? kv[(size_t)t * ldkv + (size_t)H * D + (size_t)h * V + j] : zero;
+}
+
+// The same for rows without padding (kw = D + P, vw = V) whose pieces are all multiples of 16 bytes, every row aligned: one
+// block a token, 16 bytes an access, queries left where they are (qt null) or copied.
+template <typename A>
+__global__ void __launch_bounds__(256) latent_heads_vec_kernel(const A* __restrict__ q, int ldq, const A* __restrict__ kv, int ldkv,
+                                                               const A* __restrict__ dense, int ldd, int R,
+                                                               const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
+                                                               const int* __restrict__ table, int max_pages, A* __restrict__ kt,
+                                                               A* __restrict__ vt, A* __restrict__ qt, int H, int D, int P, int V) {
+  constexpr int E = 16 / sizeof(A);               // elements an access
+  const int t = blockIdx.x, pos = tok_pos[t];
+  const int kc = (D + P) / E, dc = D / E, vc = V / E;
+  const size_t at0 = (size_t)table[(size_t)tok_seq[t] * max_pages + pos / SLLM_PAGE] * H * SLLM_PAGE + pos % SLLM_PAGE;
+  const uint4* kv4 = (const uint4*)(kv + (size_t)t * ldkv);
+  const uint4* rot4 = (const uint4*)(dense + (size_t)t * ldd + R);
+  for (int i = threadIdx.x; i < H * kc; i += blockDim.x) {
+    const int h = i / kc, c = i % kc;
+    ((uint4*)kt)[(at0 + (size_t)h * SLLM_PAGE) * kc + c] = c < dc ? kv4[h * dc + c] : rot4[c - dc];
+    if (qt) ((uint4*)qt)[(size_t)t * H * kc + i] = ((const uint4*)(q + (size_t)t * ldq))[i];
+  }
+  for (int i = threadIdx.x; i < H * vc; i += blockDim.x) {
+    const int h = i / vc, c = i % vc;
+    ((uint4*)vt)[(at0 + (size_t)h * SLLM_PAGE) * vc + c] = kv4[H * dc + i];
   }
 }
 
@@ -506,13 +532,14 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const A* __restrict_
 // scores and sums: one block per (row, group of up to 8 heads, split of the keys), a warp per head. Keys arrive in
 // tiles of 32 rows, staged in shared memory as floats once for all heads of the block; a lane scores one key of the
 // tile, softmax statistics are renewed once per tile, and the sum over the latent runs with the columns spread over
-// the lanes (NV columns a lane). Causal: keys 0 .. pos of the row's sequence. Each split leaves (max, sum, sums over
+// the lanes (NV columns a lane). Causal: keys first_seen(pos, window) .. pos of the row's sequence; tiles that lie wholly
+// before them are not touched (their pages may be gone). Each split leaves (max, sum, sums over
 // the latent) in `part` [T][H][n_split][R + 2]; the expansion merges them.
 template <typename A, int NV>
 __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restrict__ qa, const A* __restrict__ pages,
                                                           const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                                                           const int* __restrict__ block_table, int max_pages,
-                                                          float* __restrict__ part, int H, int R, int P, int n_split, int vec) {
+                                                          float* __restrict__ part, int H, int R, int P, int n_split, int window, int vec) {
   extern __shared__ __align__(16) float sm[];
   int W = R + P, Wp = W + 1;
   int t = blockIdx.x, h0 = blockIdx.y * 8, sp = blockIdx.z;
@@ -524,9 +551,10 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
   int pos = tok_pos[t];
   const int* pt = block_table + (size_t)tok_seq[t] * max_pages;
   for (int i = threadIdx.x; i < nh * W; i += nthreads) qs[i] = qa[((size_t)t * H + h0) * W + i];
-  int n_tiles = pos / 32 + 1;
+  const int first = first_seen(pos, window), tile0 = first / 32;
+  int n_tiles = pos / 32 + 1 - tile0;
   int per = (n_tiles + n_split - 1) / n_split;
-  int tile_lo = sp * per, tile_hi = min(n_tiles, tile_lo + per);
+  int tile_lo = tile0 + sp * per, tile_hi = min(tile0 + n_tiles, tile_lo + per);
   float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
   for (int i = 0; i < NV; i++) acc[i] = 0.f;
@@ -574,7 +602,8 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
     __syncthreads();
     if (!active) continue;
     float sc = -INFINITY;
-    if (lane < nk) {
+    const bool seen = lane < nk && k0 + lane >= first;       // a tile of the walk has at least one such key
+    if (seen) {
       const float* kr = Ks + lane * Wp;
       float s0 = 0.f, s1 = 0.f;
       int d = 0;
@@ -584,7 +613,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
     }
     float m_new = fmaxf(m, warp_max(sc));
     float c = expf(m - m_new);
-    float pwt = lane < nk ? expf(sc - m_new) : 0.f;
+    float pwt = seen ? expf(sc - m_new) : 0.f;
     l = l * c + warp_sum(pwt);
     m = m_new;
 #pragma unroll
@@ -617,7 +646,7 @@ template <typename A, int NV4>
 __global__ void __launch_bounds__(256) latent_attn_vec_kernel(const float* __restrict__ qa, const A* __restrict__ pages,
                                                               const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                                                               const int* __restrict__ block_table, int max_pages,
-                                                              float* __restrict__ part, int H, int R, int P, int n_split, int Wp) {
+                                                              float* __restrict__ part, int H, int R, int P, int n_split, int window, int Wp) {
   extern __shared__ __align__(16) float sm[];
   int W = R + P;
   int t = blockIdx.x, h0 = blockIdx.y * 8, sp = blockIdx.z;
@@ -629,9 +658,10 @@ __global__ void __launch_bounds__(256) latent_attn_vec_kernel(const float* __res
   int pos = tok_pos[t];
   const int* pt = block_table + (size_t)tok_seq[t] * max_pages;
   for (int i = threadIdx.x; i < nh * W; i += nthreads) qs[i] = qa[((size_t)t * H + h0) * W + i];
-  int n_tiles = pos / 32 + 1;
+  const int first = first_seen(pos, window), tile0 = first / 32;
+  int n_tiles = pos / 32 + 1 - tile0;
   int per = (n_tiles + n_split - 1) / n_split;
-  int tile_lo = sp * per, tile_hi = min(n_tiles, tile_lo + per);
+  int tile_lo = tile0 + sp * per, tile_hi = min(tile0 + n_tiles, tile_lo + per);
   float m = -INFINITY, l = 0.f, acc[NV4][4];
 #pragma unroll
   for (int i = 0; i < NV4; i++) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
@@ -671,7 +701,8 @@ __global__ void __launch_bounds__(256) latent_attn_vec_kernel(const float* __res
     __syncthreads();
     if (!active) continue;
     float sc = -INFINITY;
-    if (lane < nk) {
+    const bool seen = lane < nk && k0 + lane >= first;       // a tile of the walk has at least one such key
+    if (seen) {
       const float4* kr = (const float4*)(Ks + lane * Wp);
       float s0 = 0.f, s1 = 0.f;
 #pragma unroll 4
@@ -684,7 +715,7 @@ __global__ void __launch_bounds__(256) latent_attn_vec_kernel(const float* __res
     }
     float m_new = fmaxf(m, warp_max(sc));
     float c = expf(m - m_new);
-    float pwt = lane < nk ? expf(sc - m_new) : 0.f;
+    float pwt = seen ? expf(sc - m_new) : 0.f;
     l = l * c + warp_sum(pwt);
     m = m_new;
 #pragma unroll
@@ -714,17 +745,20 @@ __global__ void __launch_bounds__(256) latent_attn_vec_kernel(const float* __res
 
 // merge: olat[t][h] = sum_s w_s acc_s / sum_s w_s l_s, w_s = exp(m_s - max m): the splits' sums over the latent as one
 // normalised vector [R] per (row, head). The first warp weighs the splits once (a lane takes splits lane, lane + 32, ...),
-// then every thread adds its columns over the splits with loads that do not depend on one another.
+// then every thread adds its columns over the splits with loads that do not depend on one another. A `sink` (one number a
+// head, or null) joins the denominator here, once: exp(sink - max m), nothing goes to the sums.
 #define MIX_MERGE_SPLITS 64
-__global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part, float* __restrict__ olat, int R, int n_split) {
+__global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part, float* __restrict__ olat, int R, int n_split,
+                                                           const float* __restrict__ sink, int H) {
   __shared__ float w[MIX_MERGE_SPLITS];
   __shared__ float s_inv;
   size_t item = blockIdx.x;                       // t * H + h
   const float* p0 = part + item * n_split * (R + 2);
+  const float snk = sink ? sink[item % H] : -INFINITY;
   if (n_split <= MIX_MERGE_SPLITS) {
     if (threadIdx.x < 32) {
       const int lane = threadIdx.x;
-      float ms[MIX_MERGE_SPLITS / 32], ls[MIX_MERGE_SPLITS / 32], mx = -INFINITY;
+      float ms[MIX_MERGE_SPLITS / 32], ls[MIX_MERGE_SPLITS / 32], mx = snk;
 #pragma unroll
       for (int i = 0; i < MIX_MERGE_SPLITS / 32; i++) {
         int s2 = lane + 32 * i;
@@ -741,6 +775,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
         den += ws * ls[i];
       }
       for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
+      if (sink) den += expf(snk - mx);
       if (lane == 0) s_inv = 1.0f / den;
     }
     __syncthreads();
@@ -756,13 +791,14 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
     }
     return;
   }
-  float mx = -INFINITY;
+  float mx = snk;
   for (int s = 0; s < n_split; s++) mx = fmaxf(mx, p0[(size_t)s * (R + 2)]);
   float den = 0.f;
   for (int s = 0; s < n_split; s++) {
     float ms = p0[(size_t)s * (R + 2)];
     if (ms > -INFINITY) den += expf(ms - mx) * p0[(size_t)s * (R + 2) + 1];
   }
+  if (sink) den += expf(snk - mx);
   float inv = 1.0f / den;
   for (int c = threadIdx.x; c < R; c += blockDim.x) {
     float a = 0.f;
@@ -774,11 +810,13 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   }
 }
 
-// expand: maps the summed latents to the head's values: out[t][h V + v] = Wuv[h V + v] . olat[t][h]. A block takes up
-// to 8 rows of one head and four output columns, a warp a column.
+// expand: maps the summed latents to the head's values: out[t][h V + v] = Wuv[h V + v] . olat[t][h], multiplied by the
+// sigmoid of a gate logit where there is one (gate_mode 1: one a head, 2: one an element; columns of a buffer of the element
+// type). A block takes up to 8 rows of one head and four output columns, a warp a column.
 template <typename A>
 __global__ void __launch_bounds__(128) latent_expand_kernel(const float* __restrict__ olat, const A* __restrict__ wuv,
-                                                            A* __restrict__ out, int ldo, int T, int H, int V, int R) {
+                                                            A* __restrict__ out, int ldo, int T, int H, int V, int R,
+                                                            const A* __restrict__ gate, int ldg, int gate_mode) {
   extern __shared__ __align__(16) float sm[];     // [8][R]
   int h = blockIdx.y, t0 = blockIdx.x * MIX_ABSORB_ROWS;
   int n = min(MIX_ABSORB_ROWS, T - t0);
@@ -803,7 +841,10 @@ __global__ void __launch_bounds__(128) latent_expand_kernel(const float* __restr
 #pragma unroll
   for (int r = 0; r < MIX_ABSORB_ROWS; r++) acc[r] = warp_sum(acc[r]);
   if (lane == 0)
-    for (int r = 0; r < n; r++) out[(size_t)(t0 + r) * ldo + (size_t)h * V + v] = from_f32<A>(acc[r]);
+    for (int r = 0; r < n; r++) {
+      const float z = gate_mode ? to_f32(gate[(size_t)(t0 + r) * ldg + (gate_mode == 1 ? (size_t)h : (size_t)h * V + v)]) : 0.f;
+      out[(size_t)(t0 + r) * ldo + (size_t)h * V + v] = from_f32<A>(gate_mode ? acc[r] * sigmoid_f(z) : acc[r]);
+    }
 }
 
 // ------------------------------------------------------------------ the selective scan

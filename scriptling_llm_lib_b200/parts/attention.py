@@ -40,7 +40,8 @@ Five more, none in the reference. `keep_first`: the first positions of a sequenc
 true positions; the cache keeps their pages. `biases`: stored vectors added to the projected queries, keys and values
 (in the store kernel) and to the output product (`o_name`; the mixer then answers with the output and the vector, a
 `WithRowVector`, and the next reader of the stream adds both). `qk_norm` with `per="head"`: every query and key head is
-divided by its own root mean square and multiplied by a weight of one head's width, shared by the heads. `sink_value`: the
+divided by its own root mean square and multiplied by a weight of one head's width, shared by the heads; without names no
+weight multiplies it, and `after_rotation` (which takes none) norms a head once it has turned. `sink_value`: the
 same sink logit for every head as a constant instead of a stored one (0: one is added to the denominator). `value_mix`:
 layers that share a `group` mix their values with those the group's first layer projected for the same token, v <- (1 - lam)
 v + lam v_first with lam a stored number, before they are cached; the first layer's values stay at hand for the step.
@@ -68,6 +69,29 @@ from .base import MIXERS, POSITION_ENCODINGS, Folded, Mixer, PartSpec
 from .conv import CausalConv
 from .linear import Linear
 from .norm import WithRowVector
+
+
+def prompt_attention(q, gate, ctx, kpages, vpages, block_table, n_heads, n_kv, key_dim, value_dim, span, scale, tensor_cores=True,
+                     **options):
+    """Queries q [T, n_heads * key_dim] of a step that is no decode step over paged keys and values of two widths, on the
+    kernel that takes them: in bfloat16 (unless `tensor_cores` is off) the tcgen05 kernels or the mma.sync one, else the
+    generic one. `options`: softcap, sink, keep. `gate`: logits per element [T, n_heads * value_dim] or None.
+    Returns the output and whether the gate has been applied to it (some kernels do it on their way out)."""
+    k = ctx.kernels
+    attn = torch.empty((q.shape[0], n_heads * value_dim), dtype=q.dtype, device=q.device)
+    fused = gate if gate is not None and q.dtype == torch.bfloat16 and gate_aligned(gate) else None
+    tensor_cores = tensor_cores and q.dtype == torch.bfloat16
+    if tensor_cores and PrefillAttentionTC.takes(key_dim, value_dim):
+        k.prefill_attention_tc.attn(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, n_heads,
+                                    n_kv, key_dim, span, scale, ctx.err_flag, gate=fused, v_dim=value_dim, **options)
+    elif tensor_cores and PrefillAttentionMMA.takes(key_dim, value_dim):
+        k.prefill_attention_mma.attn(q, key_dim, attn, value_dim, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs,
+                                     ctx.max_new, n_heads, n_kv, key_dim, value_dim, span, scale, gate=fused, **options)
+    else:
+        fused = None
+        k.attn_paged(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, n_heads, n_kv, key_dim,
+                     span, scale, v_dim=value_dim, **options)
+    return attn, fused is not None
 
 
 class Attention(Mixer):
@@ -151,6 +175,12 @@ class Attention(Mixer):
         self.norm_per_head = self.qk_norm is not None and self.qk_norm.get("per", "projection") == "head"
         if self.qk_norm is not None and self.qk_norm.get("per", "projection") not in ("head", "projection"):
             raise ValueError(f"a query/key norm per {self.qk_norm['per']!r}; known: head, projection")
+        self.norm_after = bool(self.qk_norm and self.qk_norm.get("after_rotation"))
+        self.norm_weights = self.qk_norm is not None and self.qk_norm.get("q_name") is not None
+        if self.qk_norm is not None and not self.norm_weights and not self.norm_after:
+            raise ValueError("a query/key norm in front of the rotation has weights")
+        if self.norm_after and (not self.norm_per_head or self.norm_weights):
+            raise ValueError("a norm behind the rotation is per head and has no weight")
         if self.conv is not None and (self.norm_per_head or self.value_mix):
             raise ValueError("behind a convolution queries and keys are normed over the whole projection and values stay unmixed")
         # what the kernels for equal widths and plain windows do not know
@@ -172,7 +202,7 @@ class Attention(Mixer):
             specs.append(TensorSpec(self.sink_name, (self.n_heads,), init="bias"))
         if self.conv is not None:
             specs += self.conv.tensor_specs()
-        if self.qk_norm is not None:
+        if self.norm_weights:
             heads = (1, 1) if self.norm_per_head else (self.n_heads, self.n_kv_heads)
             specs += [TensorSpec(self.qk_norm[n], (h * self.head_dim,), init="norm_weight") for n, h in zip(("q_name", "k_name"), heads)]
         widths = dict(zip(("q_name", "k_name", "v_name", "o_name"), self.qkv.out_features[:3] + [self.hidden]))
@@ -196,7 +226,7 @@ class Attention(Mixer):
             self.mix_share = float(tensors[self.value_mix["share_name"]].float().cpu())
         if self.conv is not None:
             self.conv.bind(tensors, dtype, device)
-        if self.qk_norm is not None:
+        if self.norm_weights:
             self.q_norm_w = tensors[self.qk_norm["q_name"]].float().contiguous()
             self.k_norm_w = tensors[self.qk_norm["k_name"]].float().contiguous()
 
@@ -293,35 +323,30 @@ class Attention(Mixer):
         """The step's queries [T, n_heads * head_dim] over the cache, with everything `general` stands for; the output
         [T, n_heads * v_dim] has been multiplied by the sigmoid of `gate` (logits per element, or None)."""
         T, H, G, hd, vd, k = q.shape[0], self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, ctx.kernels
-        attn = torch.empty((T, H * vd), dtype=q.dtype, device=q.device)
         if not q.is_contiguous():
             q = q.contiguous()
         bf16 = q.dtype == torch.bfloat16
         options = dict(softcap=self.softcap, sink=self.sink, keep=self.keep_first)
-        fused_gate = gate if gate is not None and bf16 and gate_aligned(gate) else None
         pages = ctx.pages_seen(unit) if ctx.is_decode else 0
+        gated = False
         if ctx.is_decode and bf16 and DecodeKernels.general_takes(hd, vd):
+            attn = torch.empty((T, H * vd), dtype=q.dtype, device=q.device)
+            fused_gate = gate if gate is not None and gate_aligned(gate) else None
+            gated = fused_gate is not None
             n_split = DecodeKernels.general_splits(ctx.n_seqs, G, hd, vd, pages, ctx.engine.sm_count)
             scratch = torch.empty((ctx.n_seqs * H * n_split * (vd + 2),), dtype=torch.float32, device=q.device)
             k.decode.attn_decode_general(q, attn, ctx.seq_pos0, block_table, kpages, vpages, scratch, ctx.engine.tickets(ctx.n_seqs * G),
                                          ctx.n_seqs, H, G, hd, vd, self.span, self.scale, n_split, gate=fused_gate, **options)
-        elif not ctx.is_decode and bf16 and PrefillAttentionTC.takes(hd, vd):
-            k.prefill_attention_tc.attn(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, H, G,
-                                        hd, self.span, self.scale, ctx.err_flag, gate=fused_gate, v_dim=vd, **options)
-        elif not ctx.is_decode and bf16 and PrefillAttentionMMA.takes(hd, vd):
-            k.prefill_attention_mma.attn(q, hd, attn, vd, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs,
-                                         ctx.max_new, H, G, hd, vd, self.span, self.scale, gate=fused_gate, **options)
+        elif ctx.is_decode and k.attn_decode_split_takes(hd, q.stride(0), vd):
+            attn = torch.empty((T, H * vd), dtype=q.dtype, device=q.device)
+            n_split = k.attn_decode_splits(ctx.n_seqs, H, G, pages, ctx.engine.sm_count)
+            part = torch.empty((ctx.n_seqs * H * n_split * (vd + 2),), dtype=torch.float32, device=q.device) if n_split > 1 else None
+            k.attn_decode_split(q, attn, ctx.seq_pos0, block_table, kpages, vpages, part, ctx.n_seqs, H, G, hd, self.span, self.scale,
+                                n_split, v_dim=vd, **options)
         else:
-            fused_gate = None
-            if ctx.is_decode and k.attn_decode_split_takes(hd, q.stride(0), vd):
-                n_split = k.attn_decode_splits(ctx.n_seqs, H, G, pages, ctx.engine.sm_count)
-                part = torch.empty((ctx.n_seqs * H * n_split * (vd + 2),), dtype=torch.float32, device=q.device) if n_split > 1 else None
-                k.attn_decode_split(q, attn, ctx.seq_pos0, block_table, kpages, vpages, part, ctx.n_seqs, H, G, hd, self.span, self.scale,
-                                    n_split, v_dim=vd, **options)
-            else:
-                k.attn_paged(q, attn, ctx.seq_start, ctx.seq_pos0, block_table, kpages, vpages, ctx.n_seqs, ctx.max_new, H, G, hd,
-                             self.span, self.scale, v_dim=vd, **options)
-        if gate is not None and fused_gate is None:
+            attn, gated = prompt_attention(q, gate, ctx, kpages, vpages, block_table, H, G, hd, vd, self.span, self.scale,
+                                           tensor_cores=not ctx.is_decode, **options)
+        if gate is not None and not gated:
             k.gate.head_gate(attn, gate, H * vd, 1)           # "heads" of one column each
         return attn
 
@@ -364,7 +389,7 @@ class Attention(Mixer):
         else:
             k.qk_norm_store(c, q, ctx.tok_pos, ctx.tok_seq, block_table, table, kpages, vpages, self.n_heads, self.n_kv_heads,
                             self.head_dim, self.v_dim, rot, interleaved, self.q_norm_w, self.k_norm_w, eps, bias=self.in_bias,
-                            per_head=self.norm_per_head, value_mix=self._value_mix(ctx, T, x.device))
+                            per_head=self.norm_per_head, value_mix=self._value_mix(ctx, T, x.device), norm_after=self.norm_after)
         gate = y[:, qw + kw + vw:] if self.gate_name is not None else None
         if self.general:
             attn = self._attend_general(q, gate if self.gate_per == "element" else None, ctx, unit, kpages, vpages, block_table)

@@ -1,6 +1,6 @@
 """Token embedding and output head.
 
-x[i, :] = E[id_i, :], no scaling (model_f32.go:363-369); logits = n W^T with W the embedding when
+x[i, :] = E[id_i, :] (model_f32.go:363-369), which a model may scale; logits = n W^T with W the embedding when
 the head is tied (model_f32.go:147-162, :519-524). The reference skips ids outside the table and
 leaves stale data in the row; here such an id is an error before anything runs. Both are parts
 like the others, named in a layout by kind ("token_embedding", "linear_head"): a model that scales
@@ -15,10 +15,24 @@ from .base import EMBEDDINGS, HEADS, Embedding, Head, PartSpec
 from .linear import Linear
 
 
+EMBEDDING_OUTPUT = "embedding_output"     # the key of the step's embedding output among what its parts share
+
+
 class TokenEmbedding(Embedding):
-    def __init__(self, vocab: int, width: int, name: str):
+    """x = scale * E[token]. With `keep_output` the step keeps a copy of x for a part that adds it to the stream again
+    between two layers (`embedding_again`); the kernel writes both. Scale and copy are absent in the reference."""
+
+    def __init__(self, vocab: int, width: int, name: str, scale: float = 1.0, keep_output: bool = False):
         self.vocab, self.width, self.name = vocab, width, name
+        self.scale, self.keep_output = float(scale), bool(keep_output)
         self.table = None
+
+    def _copy(self, out, ctx):
+        """Where the kernel puts the copy of its rows that the step keeps (None: nobody asks for one)."""
+        if not self.keep_output:
+            return None
+        ctx.scratch[EMBEDDING_OUTPUT] = torch.empty_like(out)
+        return ctx.scratch[EMBEDDING_OUTPUT]
 
     def tensor_specs(self):
         return [TensorSpec(self.name, (self.vocab, self.width))]
@@ -31,10 +45,8 @@ class TokenEmbedding(Embedding):
 
     def forward(self, ids, ctx):
         out = torch.empty((ids.shape[0], self.width), dtype=torch.float32, device=ids.device)
-        if self.table.dtype == ctx.dtype:
-            ctx.kernels.embed_rows(ids, self.table, out, ctx.err_flag)
-        else:
-            ctx.kernels_f32.embed_rows(ids, self.table, out, ctx.err_flag)
+        k = ctx.kernels if self.table.dtype == ctx.dtype else ctx.kernels_f32
+        k.embed_rows(ids, self.table, out, ctx.err_flag, scale=self.scale, copy=self._copy(out, ctx))
         return out
 
 
@@ -66,25 +78,24 @@ class SinusoidEmbedding(TokenEmbedding):
         return out
 
 
-class PairHashEmbedding(Embedding):
-    """x = E[token] + P[r]: a second table P [buckets + 1, width] is looked up by the pair (previous token, token),
+class PairHashEmbedding(TokenEmbedding):
+    """x = scale * E[token] + P[r]: a second table P [buckets + 1, width] is looked up by the pair (previous token, token),
     r = (previous * mul_prev + token * mul_cur) mod buckets, and by its last row, r = buckets, for a sequence's first token
     (absent in the reference). The previous token of a step's first row is per-sequence state: one int32 per slot
     (`state_need`), read and then set to the run's last token by the embedding kernel itself, so prompts in portions,
     decode steps and replayed steps all find it on the device."""
 
-    def __init__(self, vocab: int, width: int, name: str, pair_name: str, buckets: int, mul_prev: int, mul_cur: int):
+    def __init__(self, vocab: int, width: int, name: str, pair_name: str, buckets: int, mul_prev: int, mul_cur: int,
+                 scale: float = 1.0, keep_output: bool = False):
+        super().__init__(vocab, width, name, scale, keep_output)
         if buckets < 1 or mul_prev < 0 or mul_cur < 0:
             raise ValueError(f"a pair table of {buckets} buckets with multipliers {mul_prev}, {mul_cur}")
-        self.vocab, self.width, self.name, self.pair_name = vocab, width, name, pair_name
+        self.pair_name = pair_name
         self.buckets, self.mul_prev, self.mul_cur = int(buckets), int(mul_prev), int(mul_cur)
-        self.table = self.pair_table = None
+        self.pair_table = None
 
     def tensor_specs(self):
         return [TensorSpec(self.name, (self.vocab, self.width)), TensorSpec(self.pair_name, (self.buckets + 1, self.width))]
-
-    def elements_read_per_step(self) -> int:
-        return 0                                    # two rows per token, not the tables
 
     def state_need(self):
         from ..cache.needs import StateNeed
@@ -99,7 +110,7 @@ class PairHashEmbedding(Embedding):
         out = torch.empty((ids.shape[0], self.width), dtype=torch.float32, device=ids.device)
         k = ctx.kernels if self.table.dtype == ctx.dtype else ctx.kernels_f32
         k.embed_pair_rows(ids, ctx, self.table, self.pair_table, self.buckets, self.mul_prev, self.mul_cur,
-                          ctx.unit_state(EMBEDDING_STATE), out, ctx.err_flag)
+                          ctx.unit_state(EMBEDDING_STATE), out, ctx.err_flag, scale=self.scale, copy=self._copy(out, ctx))
         return out
 
 
@@ -143,8 +154,13 @@ EMBEDDINGS.register("pair_hash_embedding", PairHashEmbedding)
 HEADS.register("linear_head", OutputHead)
 
 
-def token_embedding(vocab: int, width: int, name: str) -> PartSpec:
-    return PartSpec("token_embedding", dict(vocab=vocab, width=width, name=name))
+def token_embedding(vocab: int, width: int, name: str, scale: float = 1.0, keep_output: bool = False) -> PartSpec:
+    params = dict(vocab=vocab, width=width, name=name)
+    if scale != 1.0:
+        params["scale"] = scale
+    if keep_output:
+        params["keep_output"] = True
+    return PartSpec("token_embedding", params)
 
 
 def linear_head(vocab: int, width: int, weight_name: str, tied: bool = False, softcap: float | None = None,

@@ -52,7 +52,7 @@ class RMSNorm(Norm):
             ctx.kernels.gate.add_rms_normed(residual, delta.y, delta.weight, delta.eps, norm=(self.weight, self.eps, y), rows=rows,
                                             y_bias=delta.bias)
             return y
-        if isinstance(delta, WithRowVector):
+        if isinstance(delta, (WithRowVector, list, tuple)):      # several addends: the stream takes them in a pass of its own
             take_into_stream(residual, delta, ctx)
             delta = None
         ctx.kernels.add_rmsnorm(residual, delta, rows, self.weight, y, self.eps)
