@@ -581,9 +581,44 @@ def fopezen_config(z):
             "width": z["width"]}
 
 
+# The Debusun decoder (latent attention behind a window with a sink and an elementwise gate; grouped-query attention behind a
+# window with heads normed once they have turned; the Mamba-2 recurrence; square-of-relu feed-forwards; a pair-table embedding
+# that comes back before every further pass) at layer sizes that resemble real models of its kinds: heads of 128, a latent of
+# 512 (256) with 128 + 64 query/key dims a head, recurrent heads of 64 with 128 states and twice the width inside, windows of
+# 1024. w2048-g8 has latent heads of 64 + 64 dims and cuts the recurrence into eight groups, for its vectors and for its norm.
+# Four layers of which the last three are gone through twice: seven layer runs, as many as the Llama decoder beside it has layers
+# (same width, heads and window; its gated feed-forward has three matrices, so two thirds of the width give it the same FLOPs).
+DEBUSUN_SIZES = {
+    "w1024": dict(width=1024, heads=8, kv_heads=2, dim=128, vdim=128, lat_dim=128, rot_dim=64, rank=256, window=1024, ssd_head=64,
+                  state=128, ssd_groups=1, norm_groups=1, dense_ff=4096),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, lat_dim=128, rot_dim=64, rank=512, window=1024, ssd_head=64,
+                  state=128, ssd_groups=1, norm_groups=1, dense_ff=8192),
+    "w2048-g8": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, lat_dim=64, rot_dim=64, rank=512, window=1024, ssd_head=64,
+                     state=128, ssd_groups=8, norm_groups=8, dense_ff=8192),
+}
+for _z in DEBUSUN_SIZES.values():
+    _z.update(ff=-(-2 * _z["dense_ff"] // 3 // 256) * 256, groups=1)
+
+
+def debusun_config(z):
+    ff, mask = {"ff": z["dense_ff"], "kind": "dense"}, {"size": z["window"]}
+    att = {"type": "attention", "mlp": ff, "mixer": {
+        "dim": z["dim"], "heads": z["heads"], "kv_heads": z["kv_heads"], "mask": mask, "scale": z["dim"] ** -0.5, "vdim": z["vdim"],
+        "rot": {"base": 10000.0, "dims": z["dim"]}}}
+    lat = {"type": "latent_attention", "mlp": ff, "mixer": {
+        "dim": z["lat_dim"], "heads": z["heads"], "kv_rank": z["rank"], "mask": mask, "rot_dim": z["rot_dim"], "vdim": z["vdim"],
+        "rot": {"base": 10000.0, "dims": z["rot_dim"], "scaling": {"factor": 4.0, "fast": 32.0, "original": 4096, "slow": 1.0}},
+        "scale": (z["lat_dim"] + z["rot_dim"]) ** -0.5}}
+    ssd = {"type": "mamba2", "mlp": ff, "mixer": {"conv": 4, "groups": z["ssd_groups"], "heads": 2 * z["width"] // z["ssd_head"],
+                                                  "norm_groups": z["norm_groups"], "state": z["state"], "vdim": z["ssd_head"]}}
+    return {"architecture": "Debusun", "embedding": {"bigram": {"buckets": 100003, "mul_cur": 31, "mul_prev": 1009}, "scale": 8.0},
+            "layers": [lat, att, ssd, att], "loop": {"start": 1, "stop": 4, "times": 2}, "norm": {"eps": 1e-6}, "vocab": DESIGN_VOCAB,
+            "width": z["width"]}
+
+
 DESIGNS = {"sozilix": (DESIGN_SIZES, sozilix_config, 3), "muvorax": (MUVORAX_SIZES, muvorax_config, 6),
            "belasun": (BELASUN_SIZES, belasun_config, 4), "tufazen": (TUFAZEN_SIZES, tufazen_config, 6),
-           "fopezen": (FOPEZEN_SIZES, fopezen_config, 4)}
+           "fopezen": (FOPEZEN_SIZES, fopezen_config, 4), "debusun": (DEBUSUN_SIZES, debusun_config, 7)}
 
 
 def llama_like(z, max_positions, layers_per_group=3):
@@ -1477,6 +1512,178 @@ def fopezen_kernels_alone(args):
     return 0
 
 
+def debusun_kernels_alone(args):
+    """What the Debusun decoder added to the kernels, each alone at DEBUSUN_SIZES[--design-sizes or w2048] beside its like on the
+    same rows: the recurrence with one decay per head (in chunks for a prompt, walked for a decode step) beside the selective scan
+    of the same inner width and beside linear attention with as large a state per head, the norm over runs of columns beside the
+    gated row norm, latent attention behind a window with sink and gate (per head for a prompt, over the latent for a decode
+    step) beside the same without, heads normed once they have turned beside rotation and store, the scaled pair-table
+    embedding with its copy beside the plain one. A prompt of --prefill-tokens rows and a decode step of --batch rows at
+    --context; a JSON line each (CUDA events around a captured run of launches; inputs rotate through more than L2 holds
+    where they are small)."""
+    from types import SimpleNamespace
+
+    import torch
+    from scriptling_llm_lib_b200.csrc.bindings import KernelSet, PrefillAttentionTC, ProbeKernels
+    pk = peaks()
+    fma = ProbeKernels().fma_tflops()
+    z = DEBUSUN_SIZES[(args.design_sizes or "w2048").split(",")[0]]
+    dt, dev, esz = torch.bfloat16, "cuda", 2
+    ks = KernelSet(dt)
+    W, H, G, D, V, window = (z[n] for n in ("width", "heads", "kv_heads", "dim", "vdim", "window"))
+    LD, P, R = z["lat_dim"], z["rot_dim"], z["rank"]
+    SV, N, SG = z["ssd_head"], z["state"], z["ssd_groups"]
+    I, SH = 2 * W, 2 * W // SV
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+
+    def timed(launch, n_sets, reps=8):
+        torch.cuda.synchronize()
+        side = torch.cuda.Stream()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.stream(side):
+            for i in range(2):
+                launch(i % n_sets)
+            torch.cuda.synchronize()
+            with torch.cuda.graph(graph, stream=side):
+                for i in range(max(reps, n_sets)):
+                    launch(i % n_sets)
+        for _ in range(3):
+            graph.replay()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        for _ in range(5):
+            graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / (5 * max(reps, n_sets)) * 1e3
+
+    def report(name, rows, us, nbytes=None, flops=None, like=None, tensor=True):
+        rec = {"kernel": name, "rows": rows, "us": round(us, 2)}
+        if like is not None:
+            rec["like"] = like
+        if nbytes is not None:
+            rec.update(gbs=round(nbytes / us / 1e3, 1), of_hbm=round(nbytes / us / 1e3 / pk["hbm_gbs"], 3))
+        if flops is not None:
+            rec.update(tflops=round(flops / us / 1e6, 2))
+            rec.update(of_bf16=round(flops / us / 1e6 / pk["bf16_tflops"], 3)) if tensor else rec.update(of_fma=round(flops / us / 1e6 / fma, 3))
+        print(json.dumps(rec), flush=True)
+
+    err = torch.zeros(1, dtype=torch.int32, device=dev)
+    rand = lambda *shape: torch.randn(*shape, device=dev).to(dt)
+    for label in ("prompt", "decode"):
+        T, B, ctxlen = (args.prefill_tokens, 1, args.prefill_tokens) if label == "prompt" else (args.batch, args.batch, args.context)
+        pages = -(-ctxlen // 64)
+        prompt = label == "prompt"
+        ar = lambda n: torch.arange(n, dtype=torch.int32, device=dev)
+        c = SimpleNamespace(seq_start=torch.tensor([0, T], dtype=torch.int32, device=dev) if prompt else ar(B + 1), slots=ar(B), n_seqs=B,
+                            max_new=T if prompt else 1, engine=SimpleNamespace(sm_count=sms),
+                            tok_pos=ar(T) if prompt else torch.full((B,), ctxlen - 1, dtype=torch.int32, device=dev),
+                            tok_seq=torch.zeros(T, dtype=torch.int32, device=dev) if prompt else ar(B))
+        pos0 = torch.zeros(1, dtype=torch.int32, device=dev) if prompt else c.tok_pos.clone()
+        table = ar(B * pages).view(B, pages).contiguous()
+        n_sets = 4 if prompt else 24
+        # ---- the recurrence, beside the selective scan (same inner width) and linear attention (a state as large per head)
+        CW = I + 2 * SG * N
+        xbc, proj = [rand(T, CW) for _ in range(n_sets)], [rand(T, I + CW + SH) for _ in range(n_sets)]
+        hv = lambda n, v: torch.full((n,), v, device=dev)
+        st_sets = 1 if prompt else max(1, min(12, -(-200_000_000 // (B * SH * N * SV * 4))))
+        S = [torch.zeros(B + 1, SH, N, SV, device=dev) for _ in range(st_sets)]
+        yo = torch.empty(T, I, dtype=dt, device=dev)
+        wI = torch.ones(I, device=dev)
+        state_bytes = 2 * B * SH * N * SV * 4
+        row_bytes = T * (CW + 2 * I + SH) * esz
+        q = 128                                          # a row's products: state read-out and update, and half a chunk of earlier rows
+        flops = T * SH * (2 * 2 * N * SV + (q // 2) * 2 * (N + SV)) if prompt else None
+        for fold in ((False, True) if prompt else (False,)):
+            us = timed(lambda i: ks.ssd.scan(xbc[i], proj[i][:, I + CW:], hv(SH, -4.0), hv(SH, 0.5), hv(SH, 1.0), proj[i][:, :I], S[i % st_sets],
+                                             c, yo, SH, SG, SV, N, weight=wI if fold else None), n_sets)
+            report(f"ssd {SH} heads of {SV} x {N} states, {'in chunks' if prompt else 'walked'}{', half a norm' if fold else ''} ({label})", T, us,
+                   nbytes=row_bytes + state_bytes, flops=flops)
+        xz, dtr, bc = [rand(T, 2 * I) for _ in range(n_sets)], torch.randn(T, I, device=dev), rand(T, W // 16 + 32)
+        S1 = [torch.zeros(B + 1, I, 16, device=dev) for _ in range(1 if prompt else 12)]
+        a1, zi = torch.zeros(I, 16, device=dev), torch.zeros(I, device=dev)
+        us = timed(lambda i: ks.mix.selective_scan(xz[i][:, :I], dtr, zi, a1, wI, bc, W // 16, W // 16 + 16, xz[i][:, I:], S1[i % len(S1)], c, yo,
+                                                   I, 16), n_sets)
+        report(f"selective_scan inner {I}, 16 states ({label})", T, us, nbytes=T * I * (4 + 3 * esz) + 2 * B * I * 16 * 4,
+               flops=6 * T * I * 16 if prompt else None, tensor=False, like="ssd")
+        lp = [rand(T, 4 * I) for _ in range(n_sets)]
+        S2 = [torch.zeros(B + 1, I // 128, 128, 128, device=dev) for _ in range(1 if prompt else 6)]
+        o32, dec = torch.empty(T, I, device=dev), torch.full((I // 128,), 0.99, device=dev)
+        us = timed(lambda i: ks.mix.lin_attn_decay(lp[i], 0, I, 2 * I, dec, S2[i % len(S2)], c, o32, I // 128, 128, 128), n_sets)
+        report(f"lin_attn_decay {I // 128} heads of 128 x 128 ({label})", T, us, nbytes=T * I * (3 * esz + 4) + 2 * B * I * 128 * 4,
+               flops=T * I // 128 * (2 * 2 * 128 * 128 + 16 * 4 * 128) if prompt else None, tensor=False, like="ssd")
+        cw, cb = rand(CW, 4), rand(CW)
+        cst = torch.zeros(B + 1, 3, CW, device=dev)
+        us = timed(lambda i: ks.seq.causal_conv(proj[i][:, I:I + CW], cw, cst, c, xbc[i], 4, out_bias=cb, act="silu"), n_sets)
+        report(f"causal_conv {CW} channels, 4 taps ({label})", T, us, nbytes=2 * T * CW * esz + 2 * B * 3 * CW * 4)
+        us = timed(lambda i: ks.ssd.group_norm(yo, wI, yo, z["norm_groups"], 1e-6), 1)
+        report(f"group_norm {I} in {z['norm_groups']} ({label})", T, us, nbytes=2 * T * I * esz)
+        us = timed(lambda i: ks.mix.gated_row_rms(o32, xz[i][:, I:], wI, yo, 1e-6, "silu"), n_sets)
+        report(f"gated_row_rms {I} ({label})", T, us, nbytes=T * I * (4 + 2 * esz), like="group_norm")
+        # ---- latent attention
+        KD, gates, sink = LD + P, rand(T, H * V), torch.zeros(H, device=dev)
+        seen = sum(min(i + 1, window) for i in range(T)) if prompt else B * min(ctxlen, window)
+        if prompt:
+            kt, vt, qt, o = rand(pages, H, 64, KD), rand(pages, H, 64, V), rand(T, H * KD), torch.empty(T, H * V, dtype=dt, device=dev)
+            for win, full, what in ((window, True, "window, sink, gate"), (0, False, "plain")):
+                n_seen = seen if win else T * (T + 1) // 2
+                kw = dict(sink=sink, gate=gates) if full else {}
+                if PrefillAttentionTC.takes(KD, V):
+                    us = timed(lambda i: ks.prefill_attention_tc.attn(qt, o, c.seq_start, pos0, table, kt, vt, 1, T, H, H, KD, win, 0.07, err,
+                                                                      v_dim=V, **kw), 1)
+                else:
+                    us = timed(lambda i: ks.prefill_attention_mma.attn(qt, KD, o, V, c.seq_start, pos0, table, kt, vt, 1, T, H, H, KD, V, win,
+                                                                       0.07, **kw), 1)
+                report(f"prompt attention from the latent, {H} heads of {KD}/{V}, {what}", T, us, flops=2 * H * (KD + V) * n_seen,
+                       like=None if full else "window, sink, gate")
+            kv, dense, qq = rand(T, H * (LD + V)), rand(T, R + P), rand(T, H * KD + R + P)
+            us = timed(lambda i: ks.mix.latent_heads(qq[:, :H * KD], kv, dense, R, c, table, kt, vt, qt, H, LD, P, V), 1)
+            report("latent_heads (prompt)", T, us, nbytes=T * H * (4 * KD + 2 * V) * esz)
+        else:
+            latp = rand(B * pages + 1, 1, 64, R + P)
+            wuk, wuv, qq = rand(H * LD, R), rand(H * V, R), rand(T, H * KD)
+            qa, olat, ao = torch.empty(T, H, R + P, device=dev), torch.empty(T, H, R, device=dev), torch.empty(T, H * V, dtype=dt, device=dev)
+            us = timed(lambda i: ks.mix.latent_absorb(qq, wuk, qa, H, LD, P, R, 0.07), 1)
+            report("latent_absorb (decode)", T, us, nbytes=H * LD * R * esz)
+            for win, what in ((window, f"window {window}"), (0, "plain")):
+                seen_pages = min(pages, (window + 126) // 64) if win else pages
+                ns = max(1, min(-(-2 * sms // (B * -(-H // 8))), seen_pages * 2, 64))
+                part = torch.empty(T, H, ns, R + 2, device=dev)
+                us = timed(lambda i: ks.mix.latent_attn(qa, latp, c, table, part, H, R, P, ns, window=win), 1)
+                n_keys = min(ctxlen, win) if win else ctxlen
+                report(f"latent_attn rank {R} + {P}, {what}, {ns} splits (decode)", T, us, nbytes=B * n_keys * (R + P) * esz,
+                       flops=2 * B * H * n_keys * (2 * R + P), tensor=False, like=None if win else "window")
+                us = timed(lambda i: ks.mix.latent_expand(part, olat, wuv, ao, H, V, R, ns, **(dict(sink=sink, gate=gates) if win else {})), 1)
+                report(f"latent_expand, {'sink, gate' if win else 'plain'} (decode)", T, us, nbytes=H * V * R * esz + T * H * ns * R * 4,
+                       like=None if win else "sink, gate")
+        # ---- heads normed once they have turned, beside rotation and store
+        C = (H + G) * D + G * V
+        ys = [rand(T, C) for _ in range(n_sets)]
+        kp, vp, qo = rand(B * pages + 1, G, 64, D), rand(B * pages + 1, G, 64, V), torch.empty(T, H * D, dtype=dt, device=dev)
+        cs = torch.randn(ctxlen + 1, D // 2, 2, device=dev)
+        us = timed(lambda i: ks.gate.qk_norm_store(ys[i], qo, c.tok_pos, c.tok_seq, table, cs, kp, vp, H, G, D, V, D, True, None, None, 1e-6,
+                                                   per_head=True, norm_after=True), n_sets)
+        report(f"qk_norm_store, normed behind the rotation ({label})", T, us, nbytes=2 * T * C * esz)
+        if D == V:
+            us = timed(lambda i: ks.rope_kv_write(ys[i], c.tok_pos, c.tok_seq, table, cs, kp, vp, H, G, D, D, True), n_sets)
+            report(f"rope_kv_write ({label})", T, us, nbytes=2 * T * C * esz, like="qk_norm_store")
+        # ---- the embedding with its copy, beside the plain one; the sum that opens a pass, beside an ordinary norm's
+        tab, pair = rand(DESIGN_VOCAB, W), rand(100004, W)
+        tok = torch.randint(0, DESIGN_VOCAB, (T,), dtype=torch.int32, device=dev)
+        xs, copy, last = [torch.randn(T, W, device=dev) for _ in range(n_sets)], torch.empty(T, W, device=dev), torch.zeros(B + 1, dtype=torch.int32, device=dev)
+        us = timed(lambda i: ks.embed_pair_rows(tok, c, tab, pair, 100003, 1009, 31, last, xs[i], err, scale=8.0, copy=copy), n_sets)
+        report(f"embed_pair_rows with a copy ({label})", T, us, nbytes=T * W * (2 * esz + 8))
+        us = timed(lambda i: ks.embed_pair_rows(tok, c, tab, pair, 100003, 1009, 31, last, xs[i], err), n_sets)
+        report(f"embed_pair_rows ({label})", T, us, nbytes=T * W * (2 * esz + 4), like="with a copy")
+        add, vec, out, w1 = [rand(T, W) for _ in range(n_sets)], torch.randn(W, device=dev), torch.empty(T, W, dtype=dt, device=dev), torch.ones(W, device=dev)
+        us = timed(lambda i: ks.gate.add_list_cast(xs[i], [add[i], copy], None, vec), n_sets)
+        report(f"add_list_cast, an addend, the embedding and a vector ({label})", T, us, nbytes=T * W * (12 + esz))
+        us = timed(lambda i: ks.add_rmsnorm(xs[i], add[i], None, w1, out, 1e-6), n_sets)
+        report(f"add_rmsnorm ({label})", T, us, nbytes=T * W * (8 + 2 * esz), like="add_list_cast")
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1502,7 +1709,7 @@ def main():
     ap.add_argument("--no-shapes", dest="shapes", action="store_false", help="skip the Llama-3.2-1B and Llama-3.1-8B sizes")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode"],
                     help="run one part only (a small case to profile); the JSON line then holds that part alone")
-    ap.add_argument("--kernel", default=None, choices=["attn_decode", "gemm_small_m", "sequence", "mix", "gate", "tufazen", "fopezen"],
+    ap.add_argument("--kernel", default=None, choices=["attn_decode", "gemm_small_m", "sequence", "mix", "gate", "tufazen", "fopezen", "debusun"],
                     help="time one decode kernel alone at --shape, --batch (and --context) instead of the model; 'sequence': "
                          "the kernels of the mixers with state at --design-sizes, for a prompt and for a decode step; 'mix': "
                          "the same for the kernels of latent attention, decayed linear attention, the selective scan and "
@@ -1512,7 +1719,9 @@ def main():
                          "before a tanh norm, the pair-table embedding, the gate per element, the router over groups, the dense "
                          "clamped gate), each beside its like; 'fopezen': what the Fopezen decoder added (attention over a window "
                          "with kept positions, a sink and a gate, biases with query/key norm and mixed values in the store kernel, "
-                         "the normed addend with a bias and a copy, the embedding with positions, the square of relu), likewise")
+                         "the normed addend with a bias and a copy, the embedding with positions, the square of relu), likewise; "
+                         "'debusun': what the Debusun decoder added (the Mamba-2 recurrence walked and in chunks, its convolution and "
+                         "norms, latent attention behind a window with a sink and a gate, heads normed behind the rotation), likewise")
     ap.add_argument("--design", default=None, choices=sorted(DESIGNS),
                     help="measure this design's prompt step and decoding at a few real layer sizes beside the Llama decoder "
                          "of equal size (--prefill-tokens, --batch, --context, --steps, --dtype, --only apply) instead of the "
@@ -1537,6 +1746,8 @@ def main():
         return tufazen_kernels_alone(args)
     if args.kernel == "fopezen":
         return fopezen_kernels_alone(args)
+    if args.kernel == "debusun":
+        return debusun_kernels_alone(args)
     if args.kernel is not None:
         return kernel_alone(args)
     if args.design is not None:

@@ -1158,11 +1158,12 @@ class SsdKernels:
         if chunked is None:
             chunked = self.dtype == torch.bfloat16 and ctx.max_new >= self.CHUNK_MIN_ROWS
         chunked = chunked and n_state <= self.CHUNK_MAX_STATE
-        states = decays = sumsq = None
+        states = decays = sums = sumsq = None
         if chunked:
             n = T // self.CHUNK + ctx.n_seqs
             states = torch.empty((n, n_heads, n_state, head_dim), dtype=torch.float32, device=out.device)
             decays = torch.empty((n, n_heads), dtype=torch.float32, device=out.device)
+            sums = torch.empty((n, n_heads, 3, self.CHUNK), dtype=torch.float32, device=out.device)
         if weight is not None:
             sumsq = torch.empty((n_heads * -(-head_dim // (64 if chunked else 32)), T), dtype=torch.float32, device=out.device)
         _check(self._fn("ssd")(
@@ -1170,7 +1171,7 @@ class SsdKernels:
             _ptr(a_log, torch.float32, "a_log"), _ptr(dskip, torch.float32, "dskip"), self._view(z, "z"), c_int(z.stride(0)),
             _ptr(state, torch.float32, "state"), _ptr(ctx.seq_start, torch.int32, "seq_start"), _ptr(ctx.slots, torch.int32, "slots"),
             self._view(out, "out"), c_int(out.stride(0)), _ptr(weight, torch.float32, "weight"), _ptr(sumsq, torch.float32, "sumsq"),
-            _ptr(states, torch.float32, "states"), _ptr(decays, torch.float32, "decays"), c_int(ctx.n_seqs), c_int(max(1, ctx.max_new)),
+            _ptr(states, torch.float32, "states"), _ptr(decays, torch.float32, "decays"), _ptr(sums, torch.float32, "sums"), c_int(ctx.n_seqs), c_int(max(1, ctx.max_new)),
             c_int(T), c_int(n_heads), c_int(n_groups), c_int(head_dim), c_int(n_state), _stream()), "ssd")
         if chunked:
             LAUNCHES[0] += 2

@@ -264,10 +264,15 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_kernel(QkStoreAr
   }
 }
 
-// The common case of the above (no rotation, heads of up to 128 in multiples of 4, at most 8 NB query and key heads, float
-// weights): a warp's heads in one batch, and every load is asked for before the first is used; biases and weights, which no
-// kernel of a step writes, even before the wait for the kernel in front.
-template <typename A, int NB>
+// The common case of the above (heads of up to 128 in multiples of 4, at most 8 NB query and key heads, float weights; no
+// rotation, or with ROT adjacent pairs: a lane's four elements are two whole pairs, whose angles it reads once for all heads;
+// BARE: neither biases nor weights nor mixed values, which leaves room for more warps): a
+// warp's heads in one batch, and every load is asked for before the first is used; biases and weights, which no kernel of a
+// step writes, even before the wait for the kernel in front.
+__device__ __forceinline__ float4 turned(const float4& x, const float2& a, const float2& b) {
+  return make_float4(x.x * a.x - x.y * a.y, x.y * a.x + x.x * a.y, x.z * b.x - x.w * b.y, x.w * b.x + x.z * b.y);
+}
+template <typename A, int NB, bool ROT, bool BARE>
 __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_small_kernel(QkStoreArgs p) {
   __shared__ float red[2][QKS_WARPS];
   pdl_launch_dependents();
@@ -281,18 +286,24 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_small_kernel(QkS
     const int head = warp + n * QKS_WARPS;
     const bool ok = on && head < heads;
     const float* wp = (const float*)(head < H ? p.qw : p.kw);
-    b[n] = ok && p.bias ? *(const float4*)(p.bias + head * hd + j) : zero;
-    w[n] = ok && wp ? *(const float4*)(wp + (p.per_head ? j : head < H ? head * hd + j : head * hd - QW + j)) : zero;
+    b[n] = !BARE && ok && p.bias ? *(const float4*)(p.bias + head * hd + j) : zero;
+    w[n] = !BARE && ok && wp ? *(const float4*)(wp + (p.per_head ? j : head < H ? head * hd + j : head * hd - QW + j)) : zero;
   }
   const int e = threadIdx.x * 4;
-  float4 vb = p.bias && e < VW ? *(const float4*)(p.bias + QW + KW + e) : zero;
+  float4 vb = !BARE && p.bias && e < VW ? *(const float4*)(p.bias + QW + KW + e) : zero;
   pdl_wait();
   const int pos = p.tok_pos[t];
   const A* c = (const A*)p.c + (size_t)t * p.ld;
   A* vm = (A*)p.vmix + (size_t)t * VW;
 #pragma unroll
   for (int n = 0; n < NB; n++) x[n] = on && warp + n * QKS_WARPS < heads ? ld4(c + (warp + n * QKS_WARPS) * hd + j) : zero;
-  float4 v = e < VW ? ld4(c + QW + KW + e) : zero, f = p.mix_mode == 2 && e < VW ? ld4((const A*)vm + e) : zero;
+  float2 r0 = make_float2(1.f, 0.f), r1 = r0;    // (cos, sin) of the lane's pairs; those behind the rotated dims stay as they are
+  if constexpr (ROT) {
+    const float2* csr = p.cs + (size_t)pos * (p.rot >> 1) + (j >> 1);
+    if (j < p.rot) r0 = csr[0];
+    if (j + 2 < p.rot) r1 = csr[1];
+  }
+  float4 v = e < VW ? ld4(c + QW + KW + e) : zero, f = !BARE && p.mix_mode == 2 && e < VW ? ld4((const A*)vm + e) : zero;
   size_t page_slot = 0;
   if (p.G > 0) {
     const int page = p.block_table[(size_t)p.tok_seq[t] * p.max_pages + pos / SLLM_PAGE];
@@ -301,11 +312,12 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_small_kernel(QkS
   float ss[NB];
 #pragma unroll
   for (int n = 0; n < NB; n++) {
-    x[n].x += b[n].x; x[n].y += b[n].y; x[n].z += b[n].z; x[n].w += b[n].w;
+    if (!BARE) { x[n].x += b[n].x; x[n].y += b[n].y; x[n].z += b[n].z; x[n].w += b[n].w; }
+    if (ROT && p.norm_after) x[n] = turned(x[n], r0, r1);
     ss[n] = warp_sum(fmaf(x[n].x, x[n].x, fmaf(x[n].y, x[n].y, fmaf(x[n].z, x[n].z, x[n].w * x[n].w))));
   }
   float rq = 1.f, rk = 1.f;
-  if (!p.per_head && (p.qw || p.kw)) {
+  if (!BARE && !p.per_head && (p.qw || p.kw)) {
     float sq = 0.f, sk = 0.f;
 #pragma unroll
     for (int n = 0; n < NB; n++) {
@@ -323,10 +335,14 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_small_kernel(QkS
   for (int n = 0; n < NB; n++) {
     const int head = warp + n * QKS_WARPS;
     if (head < heads && on) {
-      if (head < H ? p.qw != nullptr : p.kw != nullptr) {
+      if (!BARE && (head < H ? p.qw != nullptr : p.kw != nullptr)) {
         const float r = p.per_head ? 1.0f / sqrtf(ss[n] / (float)hd + p.eps) : head < H ? rq : rk;
         x[n] = make_float4(x[n].x * r * w[n].x, x[n].y * r * w[n].y, x[n].z * r * w[n].z, x[n].w * r * w[n].w);
+      } else if (p.norm_after) {
+        const float r = 1.0f / sqrtf(ss[n] / (float)hd + p.eps);
+        x[n] = make_float4(x[n].x * r, x[n].y * r, x[n].z * r, x[n].w * r);
       }
+      if (ROT && !p.norm_after) x[n] = turned(x[n], r0, r1);
       if (head < H) st4((A*)p.q_out + (size_t)t * p.ldq + head * hd + j, x[n]);
       else st4((A*)p.kpages + (page_slot + (size_t)(head - H) * SLLM_PAGE) * hd + j, x[n]);
     }
@@ -334,12 +350,12 @@ __global__ void __launch_bounds__(QKS_WARPS * 32) qk_norm_store_small_kernel(QkS
   for (int k = e; k < VW; k += QKS_WARPS * 32 * 4) {
     if (k != e) {
       v = ld4(c + QW + KW + k);
-      if (p.bias) vb = *(const float4*)(p.bias + QW + KW + k);
-      if (p.mix_mode == 2) f = ld4((const A*)vm + k);
+      if (!BARE && p.bias) vb = *(const float4*)(p.bias + QW + KW + k);
+      if (!BARE && p.mix_mode == 2) f = ld4((const A*)vm + k);
     }
-    v.x += vb.x; v.y += vb.y; v.z += vb.z; v.w += vb.w;
-    if (p.mix_mode == 1) st4(vm + k, v);
-    if (p.mix_mode == 2) {
+    if (!BARE) { v.x += vb.x; v.y += vb.y; v.z += vb.z; v.w += vb.w; }
+    if (!BARE && p.mix_mode == 1) st4(vm + k, v);
+    if (!BARE && p.mix_mode == 2) {
       const float a = 1.0f - p.lam;
       v = make_float4(a * v.x + p.lam * f.x, a * v.y + p.lam * f.y, a * v.z + p.lam * f.z, a * v.w + p.lam * f.w);
     }

@@ -187,6 +187,79 @@ __global__ void causal_conv_vec_kernel(ConvArgs p) {
   if (p.y2) st4((A*)p.y2 + (size_t)t * p.ldy2 + c, acc);
 }
 
+// The same for steps of many rows: four neighbouring channels and ROWS rows a thread, whose inputs it reads once (all asked for
+// before the first is used) with the channels' filters in registers. TAPS: the number of taps.
+template <typename A, int TAPS, int ROWS>
+__global__ void __launch_bounds__(128) causal_conv_rows_kernel(ConvArgs p, int T) {
+  constexpr int HIST = TAPS - 1;
+  const int t0 = blockIdx.x * ROWS, c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (c >= p.C) return;
+  float4 v[HIST + ROWS];                        // rows t0 - HIST .. t0 + ROWS - 1
+#pragma unroll
+  for (int k = 0; k < HIST + ROWS; k++) {
+    const int s = t0 - HIST + k;
+    v[k] = s >= 0 && s < T ? ld4_flag<A>(p.x, p.x_f32, (size_t)s * p.ldx + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const int b0 = p.tok_seq[t0], first0 = p.seq_start[b0], end0 = p.seq_start[b0 + 1];
+  float w[4 * TAPS];                            // the four channels' taps lie one behind the other
+#pragma unroll
+  for (int m = 0; m < TAPS; m++) {
+    const float4 q = ld4_w(p.w, p.w_f32, (size_t)c * TAPS + 4 * m);
+    w[4 * m] = q.x; w[4 * m + 1] = q.y; w[4 * m + 2] = q.z; w[4 * m + 3] = q.w;
+  }
+  if (p.in_bias) {
+    const float4 ib = ld4_w(p.in_bias, p.b_f32, c);
+#pragma unroll
+    for (int k = 0; k < HIST + ROWS; k++) { v[k].x += ib.x; v[k].y += ib.y; v[k].z += ib.z; v[k].w += ib.w; }
+  }
+  const float4 ob = p.out_bias ? ld4_w(p.out_bias, p.b_f32, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  const bool inside = t0 - HIST >= first0 && t0 + ROWS <= end0;      // all of one sequence, nothing out of its state
+#pragma unroll
+  for (int r = 0; r < ROWS; r++) {
+    const int t = t0 + r;
+    if (!inside && t >= T) break;
+    float4 acc = ob;
+    if (inside) {
+#pragma unroll
+      for (int j = 0; j < TAPS; j++) {
+        const float4 q = v[r + j];
+        acc.x = fmaf(w[j], q.x, acc.x);
+        acc.y = fmaf(w[TAPS + j], q.y, acc.y);
+        acc.z = fmaf(w[2 * TAPS + j], q.z, acc.z);
+        acc.w = fmaf(w[3 * TAPS + j], q.w, acc.w);
+      }
+    } else {
+      const int b = p.tok_seq[t], first = p.seq_start[b];
+#pragma unroll
+      for (int j = 0; j < TAPS; j++) {
+        float4 q = v[r + j];
+        const int before = t - HIST + j - first;  // below 0: an input in front of the step, out of the sequence's state
+        if (before < 0) q = *(const float4*)(p.state + ((size_t)p.slots[b] * HIST + HIST + before) * p.C + c);
+        acc.x = fmaf(w[j], q.x, acc.x);
+        acc.y = fmaf(w[TAPS + j], q.y, acc.y);
+        acc.z = fmaf(w[2 * TAPS + j], q.z, acc.z);
+        acc.w = fmaf(w[3 * TAPS + j], q.w, acc.w);
+      }
+    }
+    if (p.add_input) {
+      const float4 q = v[r + HIST];
+      acc.x += q.x; acc.y += q.y; acc.z += q.z; acc.w += q.w;
+    }
+    if (p.act == 1) {
+      if (sizeof(A) == 2 && !p.y_f32) {         // on its way into a 16-bit number
+        acc.x = __fdividef(acc.x, 1.0f + __expf(-acc.x));
+        acc.y = __fdividef(acc.y, 1.0f + __expf(-acc.y));
+        acc.z = __fdividef(acc.z, 1.0f + __expf(-acc.z));
+        acc.w = __fdividef(acc.w, 1.0f + __expf(-acc.w));
+      } else {
+        acc.x = silu_f(acc.x); acc.y = silu_f(acc.y); acc.z = silu_f(acc.z); acc.w = silu_f(acc.w);
+      }
+    }
+    st4_flag<A>(p.y, p.y_f32, (size_t)t * p.ldy + c, acc);
+    if (p.y2) st4((A*)p.y2 + (size_t)t * p.ldy2 + c, acc);
+  }
+}
+
 // After the convolution of a step: the state becomes the last taps - 1 inputs of [state | step's rows].
 template <typename A>
 __global__ void conv_state_update_kernel(ConvArgs p, int n_seqs) {

@@ -35,6 +35,7 @@ struct Args {
   int T, H, G, V, N;
   float* chunk_state;                    // chunked form: [chunks][H][N][V]
   float* chunk_decay;                    // [chunks][H]
+  float* chunk_sums;                     // [chunks][H][3][SSD_Q]: step sizes; sums of a (base 2) of the chunk's rows as hi + lo
   int vec;                               // rows of xbc, their parts and V allow 16-byte accesses
 };
 
@@ -169,8 +170,8 @@ __global__ void __launch_bounds__(256) ssd_walk_kernel(Args p, int R) {
 //   S  <- exp(c_last) S + sum_j exp(c_last - c_j) dt_j B_j x_j^T.
 // x, B and C are bfloat16 as they come, so C . B is exact in a bfloat16 product with float sums. What is float (the state, and
 // everything that carries a step size or a decay) enters a product as the sum of three bfloat16 numbers (split3): 24 bits of
-// mantissa, so nothing is lost against float. c is summed in double and kept as two floats, so that differences of sums that
-// have grown large keep their digits.
+// mantissa, so nothing is lost against float. c is summed in double (times log2 e: the exponentials are of base 2) and kept as two
+// floats, so that differences of sums that have grown large keep their digits.
 #define SSD_Q 128
 #define SSD_VB 64            // value columns a block
 #define SSD_VS (SSD_VB + 8)  // padded row of a tile of them (elements)
@@ -190,73 +191,45 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const bf16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
 }
-__device__ __forceinline__ void split3(float v, bf16& a, bf16& b, bf16& c) {
-  a = __float2bfloat16_rn(v);
-  const float r = v - __bfloat162float(a);
-  b = __float2bfloat16_rn(r);
-  c = __float2bfloat16_rn(r - __bfloat162float(b));
-}
-__device__ __forceinline__ uint32_t pack2(bf16 a, bf16 b) {
-  __nv_bfloat162 v;
-  v.x = a; v.y = b;
-  return *(uint32_t*)&v;
-}
-// two neighbouring floats as three packed pairs
+// two neighbouring floats as three packed pairs of bfloat16 that add up to them
+__device__ __forceinline__ uint32_t bits(const __nv_bfloat162& v) { return *(const uint32_t*)&v; }
 __device__ __forceinline__ void split3_pair(float u, float v, uint32_t& p0, uint32_t& p1, uint32_t& p2) {
-  bf16 a0, b0, c0, a1, b1, c1;
-  split3(u, a0, b0, c0);
-  split3(v, a1, b1, c1);
-  p0 = pack2(a0, a1); p1 = pack2(b0, b1); p2 = pack2(c0, c1);
+  const __nv_bfloat162 a = __floats2bfloat162_rn(u, v);
+  u -= __low2float(a); v -= __high2float(a);
+  const __nv_bfloat162 b = __floats2bfloat162_rn(u, v);
+  u -= __low2float(b); v -= __high2float(b);
+  p0 = bits(a); p1 = bits(b); p2 = bits(__floats2bfloat162_rn(u, v));
+}
+// silu on its way into a bfloat16 number
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+// 16 bytes into shared memory without a register, or zeros
+__device__ __forceinline__ void cp16(bf16* dst, const bf16* src, bool there) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(there ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_wait() {
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
-// rows [0, SSD_Q) of `cols` columns (row stride ldx) into a tile of row stride `s`; rows from n on and columns from `cols` up
-// to `cols_p` (a multiple of 8) are zero
-__device__ __forceinline__ void stage_rows(bf16* dst, int s, const bf16* src, int ldx, int n, int cols, int cols_p, int vec) {
+// rows [0, SSD_Q) of `cols` columns (row stride ldx) into a tile of COLS columns and row stride COLS + 8; rows from n on and
+// columns from `cols` on are zero. cp_wait() and a barrier stand between this and a reader.
+template <int COLS>
+__device__ __forceinline__ void stage_rows(bf16* dst, const bf16* src, int ldx, int n, int cols, int vec) {
   if (vec) {
-    const int ch = cols_p >> 3;
-    for (int i = threadIdx.x; i < SSD_Q * ch; i += 256) {
-      const int r = i / ch, c = (i % ch) << 3;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (r < n && c < cols) v = *(const uint4*)(src + (size_t)r * ldx + c);
-      *(uint4*)(dst + r * s + c) = v;
+    constexpr int CH = COLS / 8;
+#pragma unroll
+    for (int i0 = 0; i0 < SSD_Q * CH; i0 += 256) {
+      const int i = i0 + threadIdx.x, r = i / CH, c = (i % CH) * 8;
+      const bool there = r < n && c < cols;
+      cp16(dst + r * (COLS + 8) + c, there ? src + (size_t)r * ldx + c : src, there);
     }
   } else {
-    for (int i = threadIdx.x; i < SSD_Q * cols_p; i += 256) {
-      const int r = i / cols_p, c = i % cols_p;
-      dst[r * s + c] = r < n && c < cols ? src[(size_t)r * ldx + c] : __float2bfloat16_rn(0.f);
+    for (int i = threadIdx.x; i < SSD_Q * COLS; i += 256) {
+      const int r = i / COLS, c = i % COLS;
+      dst[r * (COLS + 8) + c] = r < n && c < cols ? src[(size_t)r * ldx + c] : __float2bfloat16_rn(0.f);
     }
-  }
-}
-
-// step sizes of the chunk's rows and the running sums of a, the first warp's work (rows from n on: dt 0)
-__device__ __forceinline__ void chunk_sums(const Args& p, int row, int n, int h, float* dt_s, float* hi, float* lo) {
-  if (threadIdx.x >= 32) return;
-  constexpr int PER = SSD_Q / 32;
-  const int lane = threadIdx.x;
-  const double a = -(double)expf(p.a_log[h]);
-  const float bias = p.dt_bias[h];
-  float d[PER];
-  double c[PER], sum = 0.0;
-#pragma unroll
-  for (int k = 0; k < PER; k++) {
-    const int r = lane * PER + k;
-    d[k] = r < n ? softplus_f(to_f32(((const bf16*)p.dt)[(size_t)(row + r) * p.lddt + h]) + bias) : 0.f;
-    sum += a * (double)d[k];
-    c[k] = sum;
-  }
-  double before = sum;                   // inclusive over the lanes, then made exclusive
-#pragma unroll
-  for (int o = 1; o < 32; o <<= 1) {
-    const double u = __shfl_up_sync(0xffffffffu, before, o);
-    if (lane >= o) before += u;
-  }
-  before -= sum;
-#pragma unroll
-  for (int k = 0; k < PER; k++) {
-    const double t = before + c[k];
-    dt_s[lane * PER + k] = d[k];
-    hi[lane * PER + k] = (float)t;
-    lo[lane * PER + k] = (float)(t - (double)(float)t);
   }
 }
 
@@ -265,51 +238,106 @@ __device__ __forceinline__ void chunk_sums(const Args& p, int row, int n, int h,
 __device__ __forceinline__ size_t first_chunk(int start, int b) { return (size_t)(start / SSD_Q + b); }
 
 // U = sum_j B_j (w_j x_j)^T, w_j = exp(c_last - c_j) dt_j. A warp takes 16 state rows at a time (M) against the block's 64
-// columns; the contraction runs over the chunk's rows: both operands are read transposed from row-major tiles.
-__global__ void __launch_bounds__(256) ssd_chunk_states_kernel(Args p) {
+// columns; the contraction runs over the chunk's rows: both operands are read transposed from row-major tiles. The blocks of a
+// head's first columns also leave the chunk's step sizes and sums (base 2, as hi + lo) and its whole decay. NP: the state
+// rows rounded up to what the kernel is built for.
+template <int NP>
+__global__ void __launch_bounds__(256, 2) ssd_chunk_states_kernel(Args p) {
   extern __shared__ __align__(16) bf16 smb[];
-  __shared__ float dt_s[SSD_Q], hi[SSD_Q], lo[SSD_Q];
+  __shared__ float w_s[SSD_Q];
+  __shared__ double part_s[SSD_Q / 32];
+  constexpr int NS = NP + 8;
   const int b = blockIdx.z, start = p.seq_start[b], len = p.seq_start[b + 1] - start;
   const int r0 = blockIdx.x * SSD_Q;
   if (r0 >= len) return;
-  const int n = min(SSD_Q, len - r0), row = start + r0;
+  const int n = min(SSD_Q, len - r0), row = start + r0, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int vblocks = (p.V + SSD_VB - 1) / SSD_VB;
-  const int h = blockIdx.y / vblocks, v0 = (blockIdx.y % vblocks) * SSD_VB, g = h / (p.H / p.G);
-  const int Np = (p.N + 15) & ~15, NS = Np + 8, vn = min(SSD_VB, p.V - v0);
+  const int h = blockIdx.y / vblocks, v0 = (blockIdx.y % vblocks) * SSD_VB, g = h / (p.H / p.G), vn = min(SSD_VB, p.V - v0);
   bf16* Bs = smb;                        // [Q][NS]
   bf16* Xs = Bs + SSD_Q * NS;            // 3 x [Q][VS]
   const bf16* xbc = (const bf16*)p.xbc + (size_t)row * p.ldx;
-  chunk_sums(p, row, n, h, dt_s, hi, lo);
-  stage_rows(Bs, NS, xbc + (size_t)p.H * p.V + (size_t)g * p.N, p.ldx, n, p.N, Np, p.vec);
-  __syncthreads();
-  const float last_hi = hi[SSD_Q - 1], last_lo = lo[SSD_Q - 1];     // rows past n add nothing to the sum
   const bf16* xr = xbc + (size_t)h * p.V + v0;
-  for (int i = threadIdx.x; i < SSD_Q * (SSD_VB / 2); i += 256) {
-    const int r = i / (SSD_VB / 2), c = (i % (SSD_VB / 2)) * 2;
-    float u = 0.f, v = 0.f;
-    if (r < n && c < vn) {
-      const float w = expf((last_hi - hi[r]) + (last_lo - lo[r])) * dt_s[r];
-      if (p.vec) {
-        const __nv_bfloat162 q = *(const __nv_bfloat162*)(xr + (size_t)r * p.ldx + c);
-        u = w * __low2float(q); v = w * __high2float(q);
-      } else {
-        u = w * to_f32(xr[(size_t)r * p.ldx + c]);
-        v = c + 1 < vn ? w * to_f32(xr[(size_t)r * p.ldx + c + 1]) : 0.f;
-      }
+  const size_t chunk = first_chunk(start, b) + blockIdx.x;
+  float raw = 0.f;
+  if (tid < n) raw = to_f32(((const bf16*)p.dt)[(size_t)(row + tid) * p.lddt + h]);
+  stage_rows<NP>(Bs, xbc + (size_t)p.H * p.V + (size_t)g * p.N, p.ldx, n, p.N, p.vec);
+  constexpr int XI = SSD_Q * (SSD_VB / 8) / 256;          // eight columns of a row at a time
+  uint4 xv[XI];
+  if (p.vec) {
+#pragma unroll
+    for (int k = 0; k < XI; k++) {
+      const int i = k * 256 + tid, r = i / (SSD_VB / 8), c = (i % (SSD_VB / 8)) * 8;
+      xv[k] = r < n && c < vn ? *(const uint4*)(xr + (size_t)r * p.ldx + c) : make_uint4(0, 0, 0, 0);
     }
-    uint32_t q0, q1, q2;
-    split3_pair(u, v, q0, q1, q2);
-    *(uint32_t*)(Xs + r * SSD_VS + c) = q0;
-    *(uint32_t*)(Xs + (SSD_Q + r) * SSD_VS + c) = q1;
-    *(uint32_t*)(Xs + (2 * SSD_Q + r) * SSD_VS + c) = q2;
+  }
+  // a thread a row: its step size and the running sum of a, in double
+  double c = 0.0;
+  float d = 0.f;
+  if (tid < SSD_Q) {
+    if (tid < n) d = softplus_f(raw + p.dt_bias[h]);
+    c = -(double)expf(p.a_log[h]) * 1.4426950408889634 * (double)d;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const double u = __shfl_up_sync(0xffffffffu, c, o);
+      if (lane >= o) c += u;
+    }
+    if (lane == 31) part_s[warp] = c;
   }
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const size_t chunk = first_chunk(start, b) + blockIdx.x;
+  if (tid < SSD_Q) {
+    double last = 0.0;
+#pragma unroll
+    for (int k = 0; k < SSD_Q / 32; k++) {
+      if (k < warp) c += part_s[k];
+      last += part_s[k];
+    }
+    w_s[tid] = exp2f((float)(last - c)) * d;
+    if (v0 == 0) {
+      float* sums = p.chunk_sums + (chunk * p.H + h) * 3 * SSD_Q;
+      const float hi = (float)c;
+      sums[tid] = d;
+      sums[SSD_Q + tid] = hi;
+      sums[2 * SSD_Q + tid] = (float)(c - (double)hi);
+      if (tid == 0) p.chunk_decay[chunk * p.H + h] = exp2f((float)last);
+    }
+  }
+  __syncthreads();
+  if (p.vec) {
+#pragma unroll
+    for (int k = 0; k < XI; k++) {
+      const int i = k * 256 + tid, r = i / (SSD_VB / 8), cc = (i % (SSD_VB / 8)) * 8;
+      const float w = w_s[r];
+      const __nv_bfloat162* x2 = (const __nv_bfloat162*)&xv[k];
+      uint4 q[3];
+      uint32_t* q0 = (uint32_t*)&q[0];
+      uint32_t* q1 = (uint32_t*)&q[1];
+      uint32_t* q2 = (uint32_t*)&q[2];
+#pragma unroll
+      for (int e = 0; e < 4; e++) split3_pair(w * __low2float(x2[e]), w * __high2float(x2[e]), q0[e], q1[e], q2[e]);
+#pragma unroll
+      for (int part = 0; part < 3; part++) *(uint4*)(Xs + (part * SSD_Q + r) * SSD_VS + cc) = q[part];
+    }
+  } else {
+    for (int i = tid; i < SSD_Q * (SSD_VB / 2); i += 256) {
+      const int r = i / (SSD_VB / 2), cc = (i % (SSD_VB / 2)) * 2;
+      float u = 0.f, v = 0.f;
+      if (r < n && cc < vn) {
+        u = w_s[r] * to_f32(xr[(size_t)r * p.ldx + cc]);
+        v = cc + 1 < vn ? w_s[r] * to_f32(xr[(size_t)r * p.ldx + cc + 1]) : 0.f;
+      }
+      uint32_t q0, q1, q2;
+      split3_pair(u, v, q0, q1, q2);
+      *(uint32_t*)(Xs + r * SSD_VS + cc) = q0;
+      *(uint32_t*)(Xs + (SSD_Q + r) * SSD_VS + cc) = q1;
+      *(uint32_t*)(Xs + (2 * SSD_Q + r) * SSD_VS + cc) = q2;
+    }
+  }
+  cp_wait();
+  __syncthreads();
   float* dst = p.chunk_state + (chunk * p.H + h) * (size_t)p.N * p.V;
-  if (v0 == 0 && threadIdx.x == 0) p.chunk_decay[chunk * p.H + h] = expf(last_hi + last_lo);
   const int ksteps = (n + 15) / 16;
-  for (int mt = warp; mt < Np / 16; mt += 8) {
+  for (int mt = warp; mt < NP / 16; mt += 8) {
+    if (mt * 16 >= p.N) break;
     float acc[SSD_VB / 8][4];
 #pragma unroll
     for (int i = 0; i < SSD_VB / 8; i++) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
@@ -331,14 +359,16 @@ __global__ void __launch_bounds__(256) ssd_chunk_states_kernel(Args p) {
     const int ra = mt * 16 + (lane >> 2), rb = ra + 8;
 #pragma unroll
     for (int i = 0; i < SSD_VB / 8; i++) {
-      const int c = i * 8 + (lane & 3) * 2;
-      if (c < vn) {
-        if (ra < p.N) dst[(size_t)ra * p.V + v0 + c] = acc[i][0];
-        if (rb < p.N) dst[(size_t)rb * p.V + v0 + c] = acc[i][2];
-      }
-      if (c + 1 < vn) {
-        if (ra < p.N) dst[(size_t)ra * p.V + v0 + c + 1] = acc[i][1];
-        if (rb < p.N) dst[(size_t)rb * p.V + v0 + c + 1] = acc[i][3];
+      const int cc = i * 8 + (lane & 3) * 2;
+      if (p.vec) {
+        if (cc < vn && ra < p.N) *(float2*)(dst + (size_t)ra * p.V + v0 + cc) = make_float2(acc[i][0], acc[i][1]);
+        if (cc < vn && rb < p.N) *(float2*)(dst + (size_t)rb * p.V + v0 + cc) = make_float2(acc[i][2], acc[i][3]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+          const int r = e < 2 ? ra : rb, q = cc + (e & 1);
+          if (q < vn && r < p.N) dst[(size_t)r * p.V + v0 + q] = acc[i][e];
+        }
       }
     }
   }
@@ -359,7 +389,7 @@ __global__ void __launch_bounds__(256) ssd_chunk_pass_kernel(Args p) {
   float s[E];
 #pragma unroll
   for (int e = 0; e < E; e++) s[e] = st[e];
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 8;
   for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
     float add[AHEAD][E], d[AHEAD];
 #pragma unroll
@@ -393,62 +423,90 @@ __global__ void __launch_bounds__(256) ssd_chunk_pass_kernel(Args p) {
 // A chunk's output. A warp takes 16 of the chunk's rows (M). First C_i against the state in front of the chunk, times
 // exp(c_i); then, 16 earlier rows j at a time, the products C_i . B_j become weights in registers (the accumulators of one
 // product are the other's A operand as they stand) that meet x_j. The state's tile and the tiles of B and x share their place.
-__global__ void __launch_bounds__(256) ssd_chunk_scan_kernel(Args p) {
+template <int NP>
+__global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_scan_kernel(Args p) {
   extern __shared__ __align__(16) bf16 smb[];
-  __shared__ float dt_s[SSD_Q], hi[SSD_Q], lo[SSD_Q];
+  __shared__ __align__(16) float sums_s[3 * SSD_Q];
+  constexpr int NS = NP + 8;
   const int b = blockIdx.z, start = p.seq_start[b], len = p.seq_start[b + 1] - start;
   const int r0 = blockIdx.x * SSD_Q;
   if (r0 >= len) return;
-  const int n = min(SSD_Q, len - r0), row = start + r0;
+  const int n = min(SSD_Q, len - r0), row = start + r0, tid = threadIdx.x;
   const int vblocks = (p.V + SSD_VB - 1) / SSD_VB;
-  const int h = blockIdx.y / vblocks, v0 = (blockIdx.y % vblocks) * SSD_VB, g = h / (p.H / p.G);
-  const int Np = (p.N + 15) & ~15, NS = Np + 8, vn = min(SSD_VB, p.V - v0);
+  const int h = blockIdx.y / vblocks, v0 = (blockIdx.y % vblocks) * SSD_VB, g = h / (p.H / p.G), vn = min(SSD_VB, p.V - v0);
   bf16* Cs = smb;                        // [Q][NS]
-  bf16* Ss = Cs + SSD_Q * NS;            // 3 x [Np][VS], later
+  bf16* Ss = Cs + SSD_Q * NS;            // 3 x [NP][VS], later
   bf16* Bs = Ss;                         // [Q][NS]
   bf16* Xs = Bs + SSD_Q * NS;            // [Q][VS]
+  const float *dt_s = sums_s, *hi = sums_s + SSD_Q, *lo = sums_s + 2 * SSD_Q;
   const bf16* xbc = (const bf16*)p.xbc + (size_t)row * p.ldx;
   const bf16* bsrc = xbc + (size_t)p.H * p.V + (size_t)g * p.N;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, t = lane & 3;
+  const int warp = tid >> 5, lane = tid & 31, gr = lane >> 2, t = lane & 3;
   const size_t chunk = first_chunk(start, b) + blockIdx.x;
-  chunk_sums(p, row, n, h, dt_s, hi, lo);
-  stage_rows(Cs, NS, bsrc + (size_t)p.G * p.N, p.ldx, n, p.N, Np, p.vec);
+  const bool work = warp * 16 < n;
+  const int ia = warp * 16 + gr, ib = ia + 8;
+  stage_rows<NP>(Cs, bsrc + (size_t)p.G * p.N, p.ldx, n, p.N, p.vec);
   {
     const float* st = p.chunk_state + (chunk * p.H + h) * (size_t)p.N * p.V + v0;
-    for (int i = threadIdx.x; i < Np * (SSD_VB / 2); i += 256) {
-      const int r = i / (SSD_VB / 2), c = (i % (SSD_VB / 2)) * 2;
-      float u = 0.f, v = 0.f;
-      if (r < p.N && c < vn) {
-        if (p.vec) {
-          const float2 q = *(const float2*)(st + (size_t)r * p.V + c);
-          u = q.x; v = q.y;
-        } else {
-          u = st[(size_t)r * p.V + c];
-          v = c + 1 < vn ? st[(size_t)r * p.V + c + 1] : 0.f;
+    constexpr int SI = NP * (SSD_VB / 4) / 256, AT = SI < 8 ? SI : 8;      // four columns of a state row at a time, AT loads on their way
+    if (p.vec) {
+#pragma unroll 1
+      for (int k0 = 0; k0 < SI; k0 += AT) {
+        float4 q[AT];
+#pragma unroll
+        for (int k = 0; k < AT; k++) {
+          const int i = (k0 + k) * 256 + tid, r = i / (SSD_VB / 4), c = (i % (SSD_VB / 4)) * 4;
+          q[k] = r < p.N && c < vn ? *(const float4*)(st + (size_t)r * p.V + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < AT; k++) {
+          const int i = (k0 + k) * 256 + tid, r = i / (SSD_VB / 4), c = (i % (SSD_VB / 4)) * 4;
+          uint2 s0, s1, s2;
+          split3_pair(q[k].x, q[k].y, s0.x, s1.x, s2.x);
+          split3_pair(q[k].z, q[k].w, s0.y, s1.y, s2.y);
+          *(uint2*)(Ss + r * SSD_VS + c) = s0;
+          *(uint2*)(Ss + (NP + r) * SSD_VS + c) = s1;
+          *(uint2*)(Ss + (2 * NP + r) * SSD_VS + c) = s2;
         }
       }
-      uint32_t q0, q1, q2;
-      split3_pair(u, v, q0, q1, q2);
-      *(uint32_t*)(Ss + r * SSD_VS + c) = q0;
-      *(uint32_t*)(Ss + (Np + r) * SSD_VS + c) = q1;
-      *(uint32_t*)(Ss + (2 * Np + r) * SSD_VS + c) = q2;
+    } else {
+      for (int i = tid; i < NP * (SSD_VB / 2); i += 256) {
+        const int r = i / (SSD_VB / 2), c = (i % (SSD_VB / 2)) * 2;
+        const float u = r < p.N && c < vn ? st[(size_t)r * p.V + c] : 0.f, v = r < p.N && c + 1 < vn ? st[(size_t)r * p.V + c + 1] : 0.f;
+        uint32_t q0, q1, q2;
+        split3_pair(u, v, q0, q1, q2);
+        *(uint32_t*)(Ss + r * SSD_VS + c) = q0;
+        *(uint32_t*)(Ss + (NP + r) * SSD_VS + c) = q1;
+        *(uint32_t*)(Ss + (2 * NP + r) * SSD_VS + c) = q2;
+      }
     }
   }
+  for (int i = tid; i < 3 * SSD_Q; i += 256) sums_s[i] = p.chunk_sums[(chunk * p.H + h) * 3 * SSD_Q + i];
+  uint32_t zv[SSD_VB / 8][2];            // the gates of this lane's elements, on their way while the products run
+  if (p.vec && work) {
+    const bf16* z = (const bf16*)p.z + (size_t)row * p.ldz + (size_t)h * p.V + v0;
+#pragma unroll
+    for (int i = 0; i < SSD_VB / 8; i++) {
+      const int c = i * 8 + 2 * t;
+      zv[i][0] = c < vn && ia < n ? *(const uint32_t*)(z + (size_t)ia * p.ldz + c) : 0u;
+      zv[i][1] = c < vn && ib < n ? *(const uint32_t*)(z + (size_t)ib * p.ldz + c) : 0u;
+    }
+  }
+  cp_wait();
   __syncthreads();
   float acc[SSD_VB / 8][4];
 #pragma unroll
   for (int i = 0; i < SSD_VB / 8; i++) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-  const bool work = warp * 16 < n;
   const bf16* crow = Cs + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * NS + (lane >> 4) * 8;
-  const int ia = warp * 16 + gr, ib = ia + 8;
   const float hia = hi[ia], loa = lo[ia], hib = hi[ib], lob = lo[ib];
   if (work) {
-    for (int ks = 0; ks < Np / 16; ks++) {
+#pragma unroll 2
+    for (int ks = 0; ks < NP / 16; ks++) {
       uint32_t a[4];
       ldsm4(a, crow + ks * 16);
 #pragma unroll
       for (int part = 0; part < 3; part++) {
-        const bf16* s = Ss + (part * Np + ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * SSD_VS + (lane >> 4) * 8;
+        const bf16* s = Ss + (part * NP + ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * SSD_VS + (lane >> 4) * 8;
 #pragma unroll
         for (int nt = 0; nt < SSD_VB / 16; nt++) {
           uint32_t q[4];
@@ -458,54 +516,57 @@ __global__ void __launch_bounds__(256) ssd_chunk_scan_kernel(Args p) {
         }
       }
     }
-    const float ea = expf(hia + loa), eb = expf(hib + lob);
+    const float ea = exp2f(hia + loa), eb = exp2f(hib + lob);
 #pragma unroll
     for (int i = 0; i < SSD_VB / 8; i++) { acc[i][0] *= ea; acc[i][1] *= ea; acc[i][2] *= eb; acc[i][3] *= eb; }
   }
   __syncthreads();                       // the state's tile has been read
-  stage_rows(Bs, NS, bsrc, p.ldx, n, p.N, Np, p.vec);
-  stage_rows(Xs, SSD_VS, xbc + (size_t)h * p.V + v0, p.ldx, n, vn, SSD_VB, p.vec);
+  stage_rows<NP>(Bs, bsrc, p.ldx, n, p.N, p.vec);
+  stage_rows<SSD_VB>(Xs, xbc + (size_t)h * p.V + v0, p.ldx, n, vn, p.vec);
+  cp_wait();
   __syncthreads();
-  if (work) {
-    for (int jt = 0; jt <= warp; jt++) {
-      float gm[2][4];
+  if (!work) return;
+  for (int jt = 0; jt <= warp; jt++) {
+    float gm[2][4];
 #pragma unroll
-      for (int i = 0; i < 2; i++) gm[i][0] = gm[i][1] = gm[i][2] = gm[i][3] = 0.f;
-      const bf16* brow = Bs + (jt * 16 + (lane & 7) + (lane >> 4) * 8) * NS + ((lane >> 3) & 1) * 8;
-#pragma unroll 4
-      for (int ks = 0; ks < Np / 16; ks++) {
-        uint32_t a[4], q[4];
-        ldsm4(a, crow + ks * 16);
-        ldsm4(q, brow + ks * 16);
-        mma_bf16(gm[0], a, q[0], q[1]);
-        mma_bf16(gm[1], a, q[2], q[3]);
+    for (int i = 0; i < 2; i++) gm[i][0] = gm[i][1] = gm[i][2] = gm[i][3] = 0.f;
+    const bf16* brow = Bs + (jt * 16 + (lane & 7) + (lane >> 4) * 8) * NS + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int ks = 0; ks < NP / 16; ks++) {
+      uint32_t a[4], q[4];
+      ldsm4(a, crow + ks * 16);
+      ldsm4(q, brow + ks * 16);
+      mma_bf16(gm[0], a, q[0], q[1]);
+      mma_bf16(gm[1], a, q[2], q[3]);
+    }
+    uint32_t w[3][4];                    // the weights as A operands: halves of 8 rows j, three parts
+#pragma unroll
+    for (int half = 0; half < 2; half++) {
+      const int j = jt * 16 + half * 8 + 2 * t;
+      const float2 hj = *(const float2*)(hi + j), lj = *(const float2*)(lo + j), dj = *(const float2*)(dt_s + j);
+      float wa0 = gm[half][0] * (exp2f((hia - hj.x) + (loa - lj.x)) * dj.x), wa1 = gm[half][1] * (exp2f((hia - hj.y) + (loa - lj.y)) * dj.y);
+      float wb0 = gm[half][2] * (exp2f((hib - hj.x) + (lob - lj.x)) * dj.x), wb1 = gm[half][3] * (exp2f((hib - hj.y) + (lob - lj.y)) * dj.y);
+      if (jt == warp) {                  // the tile on the diagonal: later rows have no say
+        if (j > ia) wa0 = 0.f;
+        if (j + 1 > ia) wa1 = 0.f;
+        if (j > ib) wb0 = 0.f;
+        if (j + 1 > ib) wb1 = 0.f;
       }
-      uint32_t w[3][4];                  // the weights as A operands: halves of 8 rows j, three parts
+      split3_pair(wa0, wa1, w[0][2 * half], w[1][2 * half], w[2][2 * half]);
+      split3_pair(wb0, wb1, w[0][2 * half + 1], w[1][2 * half + 1], w[2][2 * half + 1]);
+    }
+    const bf16* xt = Xs + (jt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * SSD_VS + (lane >> 4) * 8;
 #pragma unroll
-      for (int half = 0; half < 2; half++) {
-        const int j = jt * 16 + half * 8 + 2 * t;
-        const float h0 = hi[j], l0 = lo[j], d0 = dt_s[j], h1 = hi[j + 1], l1 = lo[j + 1], d1 = dt_s[j + 1];
-        const float wa0 = j <= ia ? gm[half][0] * expf((hia - h0) + (loa - l0)) * d0 : 0.f;
-        const float wa1 = j + 1 <= ia ? gm[half][1] * expf((hia - h1) + (loa - l1)) * d1 : 0.f;
-        const float wb0 = j <= ib ? gm[half][2] * expf((hib - h0) + (lob - l0)) * d0 : 0.f;
-        const float wb1 = j + 1 <= ib ? gm[half][3] * expf((hib - h1) + (lob - l1)) * d1 : 0.f;
-        split3_pair(wa0, wa1, w[0][2 * half], w[1][2 * half], w[2][2 * half]);
-        split3_pair(wb0, wb1, w[0][2 * half + 1], w[1][2 * half + 1], w[2][2 * half + 1]);
-      }
-      const bf16* xt = Xs + (jt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * SSD_VS + (lane >> 4) * 8;
+    for (int nt = 0; nt < SSD_VB / 16; nt++) {
+      uint32_t q[4];
+      ldsm4t(q, xt + nt * 16);
 #pragma unroll
-      for (int nt = 0; nt < SSD_VB / 16; nt++) {
-        uint32_t q[4];
-        ldsm4t(q, xt + nt * 16);
-#pragma unroll
-        for (int part = 0; part < 3; part++) {
-          mma_bf16(acc[2 * nt], w[part], q[0], q[1]);
-          mma_bf16(acc[2 * nt + 1], w[part], q[2], q[3]);
-        }
+      for (int part = 0; part < 3; part++) {
+        mma_bf16(acc[2 * nt], w[part], q[0], q[1]);
+        mma_bf16(acc[2 * nt + 1], w[part], q[2], q[3]);
       }
     }
   }
-  if (!work) return;
   const float dsk = p.dskip[h];
   float ssa = 0.f, ssb = 0.f;
 #pragma unroll
@@ -519,24 +580,25 @@ __global__ void __launch_bounds__(256) ssd_chunk_scan_kernel(Args p) {
     for (int s = 0; s < 2; s++) {
       const int r = s ? ib : ia;
       if (r >= n) continue;
-      const bf16* z = (const bf16*)p.z + (size_t)(row + r) * p.ldz + col;
       bf16* o = (bf16*)p.out + (size_t)(row + r) * p.ldo + col;
-      const bf16* x = Xs + r * SSD_VS + c;
       float z0, z1 = 0.f;
       if (p.vec) {
-        const __nv_bfloat162 q = *(const __nv_bfloat162*)z;
+        const __nv_bfloat162 q = *(const __nv_bfloat162*)&zv[i][s];
         z0 = __low2float(q); z1 = __high2float(q);
       } else {
+        const bf16* z = (const bf16*)p.z + (size_t)(row + r) * p.ldz + col;
         z0 = to_f32(z[0]);
         if (two) z1 = to_f32(z[1]);
       }
-      const float u0 = fmaf(dsk, to_f32(x[0]), acc[i][2 * s]) * silu_f(z0);
-      const float u1 = two ? fmaf(dsk, to_f32(x[1]), acc[i][2 * s + 1]) * silu_f(z1) : 0.f;
+      const __nv_bfloat162 x = *(const __nv_bfloat162*)(Xs + r * SSD_VS + c);
+      const float u0 = fmaf(dsk, __low2float(x), acc[i][2 * s]) * silu_fast(z0);
+      const float u1 = two ? fmaf(dsk, __high2float(x), acc[i][2 * s + 1]) * silu_fast(z1) : 0.f;
       if (s) ssb += u0 * u0 + u1 * u1; else ssa += u0 * u0 + u1 * u1;
-      if (p.vec) *(uint32_t*)o = pack2(__float2bfloat16_rn(u0 * w0), __float2bfloat16_rn(u1 * w1));
+      const __nv_bfloat162 y = __floats2bfloat162_rn(u0 * w0, u1 * w1);
+      if (p.vec) *(__nv_bfloat162*)o = y;
       else {
-        o[0] = __float2bfloat16_rn(u0 * w0);
-        if (two) o[1] = __float2bfloat16_rn(u1 * w1);
+        o[0] = __low2bfloat16(y);
+        if (two) o[1] = __high2bfloat16(y);
       }
     }
   }
