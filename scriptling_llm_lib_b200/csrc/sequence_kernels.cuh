@@ -121,6 +121,7 @@ struct ConvArgs {
   void* y; int y_f32; int ldy;
   void* y2; int ldy2;
   int C, taps, add_input, act;
+  int own_state;                                // every sequence has one row: its state is moved on by the thread that reads it
 };
 
 template <typename A>
@@ -131,7 +132,7 @@ __global__ void causal_conv_kernel(ConvArgs p) {
   int b = p.tok_seq[t];
   int first = p.seq_start[b];
   int hist = p.taps - 1;
-  const float* st = p.state + (size_t)p.slots[b] * hist * p.C;
+  float* st = p.state + (size_t)p.slots[b] * hist * p.C;
   float ib = p.in_bias ? load_w(p.in_bias, p.b_f32, c) : 0.f;
   float acc = 0.f, cur = 0.f;
   for (int j = 0; j < p.taps; j++) {
@@ -139,6 +140,7 @@ __global__ void causal_conv_kernel(ConvArgs p) {
     float v;
     if (s >= first) v = ld_flag<A>(p.x, p.x_f32, (size_t)s * p.ldx + c) + ib;
     else v = st[(size_t)(hist + (s - first)) * p.C + c];      // s - first in [-hist, -1]
+    if (p.own_state && j > 0) st[(size_t)(j - 1) * p.C + c] = v;    // the entry behind it has not been read yet and stays
     acc += load_w(p.w, p.w_f32, (size_t)c * p.taps + j) * v;
     cur = v;
   }
@@ -159,7 +161,7 @@ __global__ void causal_conv_vec_kernel(ConvArgs p) {
   int b = p.tok_seq[t];
   int first = p.seq_start[b];
   int hist = p.taps - 1;
-  const float* st = p.state + (size_t)p.slots[b] * hist * p.C;
+  float* st = p.state + (size_t)p.slots[b] * hist * p.C;
   float4 ib = p.in_bias ? ld4_w(p.in_bias, p.b_f32, c) : make_float4(0.f, 0.f, 0.f, 0.f);
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), cur = acc;
   for (int j = 0; j < p.taps; j++) {
@@ -171,6 +173,7 @@ __global__ void causal_conv_vec_kernel(ConvArgs p) {
     } else {
       v = *(const float4*)(st + (size_t)(hist + (s - first)) * p.C + c);
     }
+    if (p.own_state && j > 0) *(float4*)(st + (size_t)(j - 1) * p.C + c) = v;
     acc.x += load_w(p.w, p.w_f32, (size_t)c * p.taps + j) * v.x;
     acc.y += load_w(p.w, p.w_f32, (size_t)(c + 1) * p.taps + j) * v.y;
     acc.z += load_w(p.w, p.w_f32, (size_t)(c + 2) * p.taps + j) * v.z;
